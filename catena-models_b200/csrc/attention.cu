@@ -1,8 +1,9 @@
 // Attention kernels: head norm + rotation + cache write, prefill attention over the step's
 // own keys, decode attention over the paged cache (split over fixed chunks, ordered merge).
 //
-// Masks: a key at position k is visible to a query at position p when k <= p and, for a
-// window W > 0, k + W > p.  Scores, softmax and the probability-value sums are float.
+// Masks: a key at position k is visible to a query at position p when k <= p and k is not before
+// first_visible(p, window): for a window W > 0, k + W > p; for W < 0, k lies in p's chunk of -W
+// positions.  Scores, softmax and the probability-value sums are float.
 #include "common.cuh"
 #include <math.h>
 
@@ -37,7 +38,8 @@ __device__ __forceinline__ float query_temperature(int pos, float coef, int ever
 // =========================================================================================
 // Head norm, rotation, cache write.  One warp per (token, head); q heads first, then k heads.
 //   qkv row: [ q: QH*HD | k: KVH*HD | v: KVH*HD | ... ]  (row stride ld)
-//   u = T((x * inv_rms(x)) * w)           when w is given (w_q for q heads, w_k for k heads)
+//   u = T((x * inv_rms(x)) * w)           when w is given (w_q for q heads, w_k for k heads); the mean of squares is
+//                                         over norm_dim channels (heads padded with zero channels: norm_dim < HD)
 //   o_i       = u_i cos a - u_{i+HD/2} sin a
 //   o_{i+HD/2}= u_{i+HD/2} cos a + u_i sin a,   a = float(pos) * rate[i]      when rate is given
 // (pairs of the two halves; with `interleaved` the pairs are neighbours, (2i, 2i+1), instead)
@@ -53,7 +55,7 @@ __global__ void qk_prepare_kernel(T* __restrict__ qkv, long long ld, const float
                                   const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                                   const int* __restrict__ seq_slot, const int* __restrict__ seq_end,
                                   T* __restrict__ pool, long long pages, const int* __restrict__ ptab,
-                                  int ptab_stride, int ring, int QH, int KVH, int HD, float eps, int T_tokens,
+                                  int ptab_stride, int ring, int QH, int KVH, int HD, int norm_dim, float eps, int T_tokens,
                                   int heads_per_warp, int interleaved, float qt_coef, int qt_every) {
     pdl_trigger();
     pdl_wait();
@@ -107,7 +109,7 @@ __global__ void qk_prepare_kernel(T* __restrict__ qkv, long long ld, const float
         float inv = 1.f;
         if (w) {
             ss = warp_sum(ss);
-            inv = 1.f / sqrtf(ss / (float)HD + eps);
+            inv = 1.f / sqrtf(ss / (float)norm_dim + eps);
         }
         T* kdst = (!is_q && page >= 0) ? kv_tile(pool, 0, pages, page, head - QH, KVH, HD) + (long long)row * HD : nullptr;
 #pragma unroll
@@ -154,7 +156,7 @@ qk_prepare_vec_kernel(T* __restrict__ qkv, long long ld, const float* __restrict
                       const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                       const int* __restrict__ seq_slot, const int* __restrict__ seq_end,
                       T* __restrict__ pool, long long pages, const int* __restrict__ ptab,
-                      int ptab_stride, int ring, int QH, int KVH, int HD, float eps, int T_tokens,
+                      int ptab_stride, int ring, int QH, int KVH, int HD, int norm_dim, float eps, int T_tokens,
                       int passes_per_warp, float qt_coef, int qt_every) {
     pdl_trigger();
     pdl_wait();
@@ -201,7 +203,7 @@ qk_prepare_vec_kernel(T* __restrict__ qkv, long long ld, const float* __restrict
         if (wq || wk) {                                             // the shuffles are for the whole warp
             float tot = 0.f;
             for (int j = 0; j < LPH; ++j) tot += __shfl_sync(0xffffffffu, ss, (hsel * LPH + j) & 31);
-            if (w) inv = 1.f / sqrtf(tot / (float)HD + eps);
+            if (w) inv = 1.f / sqrtf(tot / (float)norm_dim + eps);
         }
         if (!live) continue;
         if (w) {
@@ -251,11 +253,12 @@ extern "C" int cm_qk_prepare(int dt, void* qkv, long long ld, const float* wq, c
                              const float* rate, const int* tok_pos, const int* tok_seq,
                              const int* seq_slot, const int* seq_end, void* pool, long long pages,
                              const int* ptab, int ptab_stride, int ring, int T, int QH, int KVH,
-                             int HD, float eps, int interleaved, float qt_coef, int qt_every, cudaStream_t st) {
+                             int HD, int norm_dim, float eps, int interleaved, float qt_coef, int qt_every, cudaStream_t st) {
     if (T <= 0) return CM_OK;
     if (HD % 2 || HD <= 0) CM_REFUSE("qk_prepare: head size %d is not even", HD);
     if (ring % PAGE_TOKENS) CM_REFUSE("qk_prepare: ring of %d entries is no multiple of %d", ring, PAGE_TOKENS);
     if (HD > CM_MAX_HEAD_DIM) CM_REFUSE("qk_prepare: head size %d above %d", HD, CM_MAX_HEAD_DIM);
+    if (norm_dim < 1 || norm_dim > HD) CM_REFUSE("qk_prepare: a norm over %d of %d channels", norm_dim, HD);
     const size_t esz = dt == DT_F32 ? 4 : 2;
     const bool vec = HD % 16 == 0 && (ld * esz) % 16 == 0 &&
                      (((uintptr_t)qkv | (uintptr_t)pool | (uintptr_t)wq | (uintptr_t)wk) & 15) == 0;
@@ -270,10 +273,10 @@ extern "C" int cm_qk_prepare(int dt, void* qkv, long long ld, const float* wq, c
         dim3 vblock(32, 4), vgrid((T + 3) / 4, (passes + ppw - 1) / ppw);
         if (dt == DT_F32)
             cm_launch(qk_prepare_vec_kernel<float>, vgrid, vblock, 0, st, (float*)qkv, ld, wq, wk, rate, tok_pos, tok_seq,
-                      seq_slot, seq_end, (float*)pool, pages, ptab, ptab_stride, ring, QH, KVH, HD, eps, T, ppw, qt_coef, qt_every);
+                      seq_slot, seq_end, (float*)pool, pages, ptab, ptab_stride, ring, QH, KVH, HD, norm_dim, eps, T, ppw, qt_coef, qt_every);
         else
             cm_launch(qk_prepare_vec_kernel<bf16>, vgrid, vblock, 0, st, (bf16*)qkv, ld, wq, wk, rate, tok_pos, tok_seq,
-                      seq_slot, seq_end, (bf16*)pool, pages, ptab, ptab_stride, ring, QH, KVH, HD, eps, T, ppw, qt_coef, qt_every);
+                      seq_slot, seq_end, (bf16*)pool, pages, ptab, ptab_stride, ring, QH, KVH, HD, norm_dim, eps, T, ppw, qt_coef, qt_every);
         CM_CHECK_LAUNCH();
         return CM_OK;
     }
@@ -283,11 +286,11 @@ extern "C" int cm_qk_prepare(int dt, void* qkv, long long ld, const float* wq, c
     if (dt == DT_F32)
         cm_launch(qk_prepare_kernel<float>, grid, block, smem, st, (float*)qkv, ld, wq, wk, rate, tok_pos, tok_seq,
                                                             seq_slot, seq_end, (float*)pool, pages, ptab,
-                                                            ptab_stride, ring, QH, KVH, HD, eps, T, hpw, interleaved, qt_coef, qt_every);
+                                                            ptab_stride, ring, QH, KVH, HD, norm_dim, eps, T, hpw, interleaved, qt_coef, qt_every);
     else if (dt == DT_BF16)
         cm_launch(qk_prepare_kernel<bf16>, grid, block, smem, st, (bf16*)qkv, ld, wq, wk, rate, tok_pos, tok_seq,
                                                            seq_slot, seq_end, (bf16*)pool, pages, ptab,
-                                                           ptab_stride, ring, QH, KVH, HD, eps, T, hpw, interleaved, qt_coef, qt_every);
+                                                           ptab_stride, ring, QH, KVH, HD, norm_dim, eps, T, hpw, interleaved, qt_coef, qt_every);
     else
         return CM_ERR_DTYPE;
     CM_CHECK_LAUNCH();
@@ -351,7 +354,7 @@ attn_prefill_simt_kernel(T* __restrict__ ctx, long long ldc, const T* __restrict
         for (int j = 0; j < AP_MAXJ; ++j) acc[i][j] = 0.f;
     }
     const int q_last = q0 + nq - 1;
-    const int k_first = window > 0 ? max(0, q0 - window + 1) : 0;    // the first key any query of the block sees
+    const int k_first = first_visible(q0, window);                   // the first key any query of the block sees
     const int k_begin = k_first / AP_BK * AP_BK;
     const int nj = (HD + 31) / 32;
 
@@ -390,7 +393,7 @@ attn_prefill_simt_kernel(T* __restrict__ ctx, long long ldc, const T* __restrict
             float s = 0.f;
             for (int d = 0; d < HD; ++d) s = fmaf(qr[d], kr[d], s);
             s = soft_cap(s * scale, cap);
-            const bool vis = qi < nq && kpos <= qpos && kpos < len && (window <= 0 || kpos + window > qpos);
+            const bool vis = qi < nq && kpos <= qpos && kpos < len && kpos >= first_visible(qpos, window);
             s = vis ? s : -INFINITY;
             const float mx = fmaxf(m[i], warp_max(s));
             float p = 0.f, alpha = 1.f;
@@ -563,6 +566,7 @@ attn_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml, cons
     const int G = QH / KVH;
     const int pos = seq_pos[b];                     // position of the query token
     const int n_entries = ring ? min(pos + 1, ring) : pos + 1;
+    const int first = first_visible(pos, window);
     const int e0 = c * AD_CHUNK;
     if (e0 >= n_entries) return;
     const int slot = seq_slot[b];
@@ -612,7 +616,7 @@ attn_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml, cons
                             if (back < 0) back += ring;
                             kpos = pos - back;
                         }
-                        v_u = kpos >= 0 && kpos <= pos && (window <= 0 || kpos + window > pos);
+                        v_u = kpos >= first && kpos <= pos;
                     }
                     if (v_u) {
                         vis_mask |= 1u << u;
@@ -654,7 +658,7 @@ attn_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml, cons
                     if (back < 0) back += ring;
                     kpos = pos - back;
                 }
-                vis = kpos >= 0 && kpos <= pos && (window <= 0 || kpos + window > pos);
+                vis = kpos >= first && kpos <= pos;
                 if (vis) {
                     const T* kr = kv_tile(pool, 0, pages, page, hk, KVH, HD) + (long long)row * HD;
                     for (int d = 0; d < HD; d += 8) {

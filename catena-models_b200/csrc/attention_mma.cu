@@ -82,7 +82,7 @@ attn_prefill_mma_kernel(bf16* __restrict__ ctx, long long ldc, const bf16* __res
     if (q0 >= len) return;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
 
-    const int k_first = window > 0 ? max(0, q0 - window + 1) : 0;   // the first key a query of this block sees
+    const int k_first = first_visible(q0, window);                  // the first key a query of this block sees
     const int kt_begin = k_first / FA_BK;
     const int kt_end = min(q0 + BQ - 1, len - 1) / FA_BK;  // inclusive
     const int* prow = PAST ? ptab + (long long)seq_slot[b] * ptab_stride : nullptr;
@@ -155,6 +155,9 @@ attn_prefill_mma_kernel(bf16* __restrict__ ctx, long long ldc, const bf16* __res
         for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
     const int row_lo = q0 + warp * 16 + g;        // this thread's rows: row_lo and row_lo + 8
+    // the first keys that they see, and those of the warp's first and last row
+    const int see[2] = {first_visible(row_lo, window), first_visible(row_lo + 8, window)};
+    const int see_first = first_visible(q0 + warp * 16, window), see_last = first_visible(q0 + warp * 16 + 15, window);
 
     for (int kt = kt_begin; kt <= kt_end; ++kt) {
         const int buf = (kt - kt_begin) & 1;
@@ -170,7 +173,7 @@ attn_prefill_mma_kernel(bf16* __restrict__ ctx, long long ldc, const bf16* __res
         const int key0 = kt * FA_BK;
         // a tile that none of this warp's 16 rows can see (all of it after them, or all of it
         // before their windows) is only waited for
-        if (key0 > q0 + warp * 16 + 15 || (window > 0 && key0 + FA_BK - 1 + window <= q0 + warp * 16)) {
+        if (key0 > q0 + warp * 16 + 15 || key0 + FA_BK - 1 < see_first) {
             __syncthreads();
             continue;
         }
@@ -212,7 +215,7 @@ attn_prefill_mma_kernel(bf16* __restrict__ ctx, long long ldc, const bf16* __res
         }
         // ---- mask, running maximum
         const bool edge = key0 + FA_BK - 1 > q0 + warp * 16 || key0 + FA_BK > len ||
-                          (window > 0 && key0 + window <= q0 + warp * 16 + 15);
+                          key0 < see_last;
         // raw scores stay unscaled; the scale (times log2 e) is folded into the exponent's argument
         float mx[2] = {-INFINITY, -INFINITY};
         if (edge) {
@@ -222,7 +225,7 @@ attn_prefill_mma_kernel(bf16* __restrict__ ctx, long long ldc, const bf16* __res
                 for (int i = 0; i < 4; ++i) {
                     const int key = key0 + 8 * j + 2 * t + (i & 1);
                     const int row = row_lo + (i >> 1) * 8;
-                    const bool vis = key <= row && key < len && (window <= 0 || key + window > row);
+                    const bool vis = key <= row && key < len && key >= see[i >> 1];
                     s[j][i] = vis ? s[j][i] : -INFINITY;
                 }
         }
@@ -437,8 +440,20 @@ attn_decode_mma_kernel(float* __restrict__ part_o, float* __restrict__ part_ml, 
     bf16* Ks = kv_s + (size_t)warp * 2 * FD_PAGE * LDS;
     bf16* Vs = Ks + FD_PAGE * LDS;
     const int* my_ptab = ptab + (long long)slot * ptab_stride;
-    // every full page is wholly visible unless the ring is wider than the window
-    const bool mask_all = window > 0 && ring != window;
+    // every full page is wholly visible unless the ring is wider than the window, or the mask goes by chunks
+    const bool mask_all = window < 0 || (window > 0 && ring != window);
+    const int first = first_visible(pos, window);
+    // This warp's next page from `idx` on that holds a visible position.  The page of the newest entry does; another page's
+    // last position is that of the newest entry less their distance (plus, behind it, a turn of the ring).
+    const int newest = ring ? pos % ring : pos;
+    auto next_page = [&](int idx) {
+        while (idx * FD_PAGE < n_entries) {
+            const int last = idx * FD_PAGE + FD_PAGE - 1;
+            if (idx == newest / FD_PAGE || pos - newest + last - (last > newest ? ring : 0) >= first) break;
+            idx += page_step;
+        }
+        return idx;
+    };
 
     // one of a page's two halves (which: 0 keys, 1 values) into this warp's buffer
     auto request = [&](bf16* dst, int which, int page_idx) {
@@ -460,7 +475,7 @@ attn_decode_mma_kernel(float* __restrict__ part_o, float* __restrict__ part_ml, 
         for (int j = 0; j < HD / 8; ++j)
 #pragma unroll
             for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
-        int page_idx = c * 4 + warp;
+        int page_idx = next_page(c * 4 + warp);
         bool live = page_idx * FD_PAGE < n_entries;
         if (live) request(Ks, 0, page_idx);
         cp_async_commit();
@@ -480,7 +495,7 @@ attn_decode_mma_kernel(float* __restrict__ part_o, float* __restrict__ part_ml, 
             }
         }
         while (live) {
-            const int next_idx = page_idx + page_step;
+            const int next_idx = next_page(page_idx + page_step);
             const bool next_live = next_idx * FD_PAGE < n_entries;
             cp_async_wait<1>();                                // this page's keys are here; its values may not be
             __syncwarp();
@@ -534,7 +549,7 @@ attn_decode_mma_kernel(float* __restrict__ part_o, float* __restrict__ part_ml, 
                                 if (back < 0) back += ring;
                                 kpos = pos - back;
                             }
-                            vis = kpos >= 0 && kpos <= pos && (window <= 0 || kpos + window > pos);
+                            vis = kpos >= first && kpos <= pos;
                         }
                         s[j][i] = vis ? s[j][i] : -INFINITY;
                     }

@@ -188,12 +188,12 @@ __device__ __forceinline__ void ft_item(int w, int tiles_x, int QH, int KVH, int
     it.p0 = 0;
     it.kt_begin = it.tp_begin = it.n_past = 0;
     if (it.q0 >= it.len) return;
-    it.kt_begin = window > 0 ? max(0, it.q0 - window + 1) / FT_TILE : 0;
-    const int kt_end = min(it.q0 + FT_TILE - 1, it.len - 1) / FT_TILE;   // inclusive
     // positions: row r of this step stands at p0 + r; tiles of the cache come first, in steps of 128 positions
     it.p0 = PAST ? past.seq_pos0[it.b] : 0;
+    const int a_lo = first_visible(it.p0 + it.q0, window);
+    it.kt_begin = max(0, a_lo - it.p0) / FT_TILE;
+    const int kt_end = min(it.q0 + FT_TILE - 1, it.len - 1) / FT_TILE;   // inclusive
     if (PAST && it.p0 > 0) {
-        const int a_lo = window > 0 ? max(0, it.p0 + it.q0 - window + 1) : 0;
         if (a_lo < it.p0) {
             it.tp_begin = a_lo / FT_TILE;
             it.n_past = (it.p0 - 1) / FT_TILE - it.tp_begin + 1;
@@ -529,7 +529,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                     }
                 }
                 // the keys of the tile that this row sees are the columns lo .. hi - 1; all of them: no comparisons needed
-                const int lo = window > 0 ? max(0, row - window + 1 - k0) : 0;
+                const int lo = max(0, first_visible(row, window) - k0);
                 const int hi = min(FT_TILE, min(row, limit - 1) - k0 + 1);
                 if (lo > 0 || hi < FT_TILE) {
                     const unsigned span = (unsigned)max(hi - lo, 0);

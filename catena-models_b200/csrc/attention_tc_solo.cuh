@@ -295,7 +295,7 @@ attn_prefill_tc_solo_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     }
                 }
                 // the keys of the tile that this row sees are the columns lo .. hi - 1; all of them: no comparisons needed
-                const int lo = window > 0 ? max(0, row - window + 1 - k0) : 0;
+                const int lo = max(0, first_visible(row, window) - k0);
                 const int hi = min(FT_TILE, min(row, limit - 1) - k0 + 1);
                 if (lo > 0 || hi < FT_TILE) {
                     const unsigned span = (unsigned)max(hi - lo, 0);

@@ -154,6 +154,16 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
     return t;
 }
 
+// The first position that a query at `pos` sees of its sequence, by the mask that the attention kernels take as one
+// number: window > 0, the last `window` positions; window < 0, the query's chunk, chunks of -window positions counted
+// from the sequence's start; 0, every earlier position.  It never falls as `pos` rises, so what a tile of queries can
+// see begins at the answer for its first row.
+__host__ __device__ __forceinline__ int first_visible(int pos, int window) {
+    if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
+    if (window < 0) return pos - pos % -window;
+    return 0;
+}
+
 // A score bounded to (-cap, cap): cap * tanh(s / cap); cap <= 0 leaves it as it is.
 __device__ __forceinline__ float soft_cap(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 // tanh from one exponential and one division (absolute error of a few 2^-24: for kernels that form

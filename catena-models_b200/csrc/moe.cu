@@ -5,7 +5,8 @@
 // routing it reads from device memory, so a step of given shape launches the same kernels with the same
 // arguments whatever the router decides, and can be recorded into a graph.
 //
-//   scores      s = gate(W_r h) in float (gate: sigmoid or softmax over the experts);
+//   scores      s = gate(W_r h (+ b)) in float (gate: sigmoid, softmax over the experts, or the logits as they are, whose
+//               softmax over the chosen ones alone gives the weights);
 //               the `top` largest, lowest index first among equals; weights = the chosen scores,
 //               optionally divided by their sum
 //   experts     a = act(W_gate x) * (W_up x), y = W_down a, with x = weight * h (the weight on the
@@ -27,7 +28,9 @@
 // ------------------------------------------------------------------------------ routing
 // How a token's experts are chosen from its E router logits, and what their weights are.
 struct RouteRule {
-    int softmax_gate;          // scores: softmax over the experts (1) or a sigmoid of each logit (0)
+    int gate;                  // scores: a sigmoid of each logit (0), a softmax over the experts (1), or the logits themselves (2);
+                               // with 2 the weights are a softmax over the chosen experts' logits alone
+    const float* bias;         // null, or [E]: added to the logits
     int renormalize;           // weights divided by (their sum + renorm_eps)
     float renorm_eps;
     float scale;               // factor on the weights
@@ -41,7 +44,11 @@ struct RouteRule {
 // One thread's walk for one token.  sc [E]: logits in, scores out (overwritten).  ch: [E] scratch for the choice scores when
 // the rule has a correction or groups, else the same array as sc.  Writes ids and wts [top]; counts every chosen real expert.
 __device__ void choose_experts(float* sc, float* ch, int E, int top, const RouteRule& r, int* ids, float* wts, int* counts) {
-    if (r.softmax_gate) {
+    if (r.bias)
+        for (int e = 0; e < E; ++e) sc[e] += r.bias[e];
+    if (r.gate == 2) {
+        // the logits are the scores
+    } else if (r.gate == 1) {
         float mx = -INFINITY, den = 0.f;
         for (int e = 0; e < E; ++e) mx = fmaxf(mx, sc[e]);
         for (int e = 0; e < E; ++e) den += expf(sc[e] - mx);
@@ -102,7 +109,12 @@ __device__ void choose_experts(float* sc, float* ch, int E, int top, const Route
         ch[best] = -INFINITY;
         if (best < r.real) atomicAdd(counts + best, 1);
     }
-    if (r.renormalize)
+    if (r.gate == 2) {
+        float mx = -INFINITY, den = 0.f;
+        for (int j = 0; j < top; ++j) mx = fmaxf(mx, wts[j]);
+        for (int j = 0; j < top; ++j) den += expf(wts[j] - mx);
+        for (int j = 0; j < top; ++j) wts[j] = expf(wts[j] - mx) / den;
+    } else if (r.renormalize)
         for (int j = 0; j < top; ++j) wts[j] /= total + r.renorm_eps;
     if (r.scale != 1.f)
         for (int j = 0; j < top; ++j) wts[j] *= r.scale;
@@ -299,13 +311,14 @@ static int max_tiles_for(long long pairs, int E, int tile_rows) {
 // E counts every router output; the last `identity` of them are identity experts (no matrices, no rows: their pairs get
 // dest -1 and a weight, see cm_moe_identity).  correction (or null), groups, keep, scale, renorm_eps: see RouteRule.
 extern "C" int cm_moe_route(int dt, int* ids, float* wts, int* perm, int* dest, int* work, const void* h, const void* wr,
-                            const int* tok_seq, long long rows, int W, int E, int top, int softmax_gate,
+                            const int* tok_seq, long long rows, int W, int E, int top, int gate,
                             int renormalize, int tile_rows, void* xs, int apply_weight, const float* correction, int groups,
-                            int keep, int identity, float scale, float renorm_eps, int group_best, cudaStream_t st) {
+                            int keep, int identity, float scale, float renorm_eps, int group_best, const float* bias, cudaStream_t st) {
     if (rows <= 0) return CM_OK;
     if (groups > 0 && (group_best < 1 || E / groups > 64 && group_best > 1))
         CM_REFUSE("moe_route: the sum of the %d best of a group of %d experts", group_best, E / groups);
     if (top < 1 || top > E) CM_REFUSE("moe_route: %d of %d experts", top, E);
+    if (gate < 0 || gate > 2) CM_REFUSE("moe_route: gate %d (0 sigmoid, 1 softmax, 2 softmax over the chosen)", gate);
     if (identity < 0 || identity >= E) CM_REFUSE("moe_route: %d identity experts of %d", identity, E);
     if (groups < 0 || groups > MOE_MAX_GROUPS || (groups > 0 && (E % groups || keep < 1 || keep > groups || keep * (E / groups) < top)))
         CM_REFUSE("moe_route: %d groups of which %d stay open, for %d of %d experts", groups, keep, top, E);
@@ -313,7 +326,8 @@ extern "C" int cm_moe_route(int dt, int* ids, float* wts, int* perm, int* dest, 
     if ((size_t)E * sizeof(float) * (two ? 2 : 1) > 48 * 1024) CM_REFUSE("moe_route: %d experts", E);
     if (tile_rows != MOE_TM && tile_rows != 128) CM_REFUSE("moe_route: row tiles of %d (32 or 128)", tile_rows);
     RouteRule rule;
-    rule.softmax_gate = softmax_gate;
+    rule.gate = gate;
+    rule.bias = bias;
     rule.renormalize = renormalize;
     rule.renorm_eps = renorm_eps;
     rule.scale = scale;

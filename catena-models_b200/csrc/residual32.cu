@@ -3,40 +3,35 @@
 // the norm of whatever runs next, and the concatenation [x; x0] that a looped stack feeds to the
 // projection at the start of a pass.
 //
-// The norm is a root-mean-square norm (kind 0) or a dynamic tanh (kind 1: y = tanh(alpha x) * w + b, which takes
-// no statistics of the row; alpha is read from the device).
+// The norm is a root-mean-square norm (kind 0), a dynamic tanh (kind 1: y = tanh(alpha x) * w + b, which takes
+// no statistics of the row; alpha is read from the device) or a layer norm without a shift (kind 2: y = (x - mean) /
+// sqrt(variance + eps) * w, the variance being the mean of the squared distances from the mean).
 //
 // A row is held in shared memory between the two passes over it (sum of squares, then scaling), so the
 // width is bounded by shared memory only.  All sums are float and run in a fixed order.
 #include "common.cuh"
+#include "residual_terms.cuh"
 
 #define R32_THREADS 256
-#define R32_MAX_TERMS 4
-
-// One term of a residual sum: rows of `per_row` consecutive pieces each (a routed feed-forward leaves
-// one piece per chosen expert), stored as float or as activations, times a constant.
-struct ResidualTerm {
-    const void* p;
-    const int* index;      // null: piece j of row r is row r * per_row + j; else row index[r * per_row + j] (negative: none)
-    const float* weights;  // null, or a factor per piece: weights[r * per_row + j] (a routed feed-forward's weights on its experts' outputs)
-    float scale;
-    int per_row;
-    int is_f32;
-};
-struct ResidualTerms {
-    ResidualTerm t[R32_MAX_TERMS];
-    int n;
-};
-
-template <typename T>
-__device__ __forceinline__ float term_at(const ResidualTerm& t, long long i) {
-    return t.is_f32 ? reinterpret_cast<const float*>(t.p)[i] : to_f32(reinterpret_cast<const T*>(t.p)[i]);
-}
-
 #define NORM_RMS 0
 #define NORM_DYT 1
+#define NORM_LAYER 2
 
-// y = T((x * inv) * w), inv = 1 / sqrt(mean(x^2) + eps); or T(tanh(alpha x) * w + b); x float.
+// A staged row moved to mean zero (`sum`: this thread's share of the row's sum; every thread touches its own columns
+// only), and the sum of the squares of what is left.
+__device__ __forceinline__ float centre_row(float* row, int H, float sum, float* scratch) {
+    const float mean = block_sum(sum, scratch) / (float)H;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        const float d = row[c] - mean;
+        row[c] = d;
+        ss += d * d;
+    }
+    return block_sum(ss, scratch);
+}
+
+// y = T((x * inv) * w), inv = 1 / sqrt(mean(x^2) + eps) (layer norm: of the row moved to mean zero); or
+// T(tanh(alpha x) * w + b); x float.
 template <typename T>
 __global__ void __launch_bounds__(R32_THREADS)
 norm_f32in_kernel(T* __restrict__ y, const float* __restrict__ x, const float* __restrict__ w, int H, float eps,
@@ -52,35 +47,18 @@ norm_f32in_kernel(T* __restrict__ y, const float* __restrict__ x, const float* _
         for (int c = threadIdx.x; c < H; c += R32_THREADS) yd[c] = from_f32<T>(fmaf(tanhf(al * xr[c]), w[c], shift[c]));
         return;
     }
-    float ss = 0.f;
+    float ss = 0.f, sum = 0.f;
     for (int c = threadIdx.x; c < H; c += R32_THREADS) {
         const float v = xr[c];
         row[c] = v;
         ss += v * v;
+        sum += v;
     }
-    ss = block_sum(ss, scratch);
+    if (kind == NORM_LAYER) ss = centre_row(row, H, sum, scratch);
+    else ss = block_sum(ss, scratch);
     const float inv = 1.f / sqrtf(ss / (float)H + eps);
     T* yr = y + (long long)blockIdx.x * H;
     for (int c = threadIdx.x; c < H; c += R32_THREADS) yr[c] = from_f32<T>((row[c] * inv) * w[c]);
-}
-
-// sum_i scale_i * sum_j (weights_i[j]) term_i[row * per_row_i + j] at column c: the terms are added to each other in their order.
-template <typename T>
-__device__ __forceinline__ float terms_at(const ResidualTerms& terms, long long r, int H, int c) {
-    float add = 0.f;
-    for (int i = 0; i < terms.n; ++i) {
-        const ResidualTerm& t = terms.t[i];
-        float s = 0.f;
-        for (int j = 0; j < t.per_row; ++j) {
-            const long long piece = t.index ? t.index[r * t.per_row + j] : r * t.per_row + j;
-            if (piece >= 0) {
-                const float v = term_at<T>(t, piece * H + c);
-                s = t.weights ? fmaf(t.weights[r * t.per_row + j], v, s) : s + v;
-            }
-        }
-        add += t.scale * s;
-    }
-    return add;
 }
 
 // h += sum_i scale_i * sum_j term_i[row * per_row_i + j] (+ bias);  n = T(norm(h) * w) when n is given.
@@ -96,13 +74,14 @@ residual_add_norm_kernel(float* __restrict__ h, T* __restrict__ n_out, ResidualT
     pdl_wait();
     const long long r = blockIdx.x;
     float* hr = h + r * H;
-    float ss = 0.f;
+    float ss = 0.f, sum = 0.f;
     for (int c = threadIdx.x; c < H; c += R32_THREADS) {
         float v = hr[c] + terms_at<T>(terms, r, H, c);
         if (bias) v += bias[c];
         hr[c] = v;
         row[c] = v;
         ss += v * v;
+        sum += v;
     }
     if (!n_out) return;
     T* nr = n_out + r * H;
@@ -111,7 +90,8 @@ residual_add_norm_kernel(float* __restrict__ h, T* __restrict__ n_out, ResidualT
         for (int c = threadIdx.x; c < H; c += R32_THREADS) nr[c] = from_f32<T>(fmaf(tanhf(al * row[c]), w[c], shift[c]));
         return;
     }
-    ss = block_sum(ss, scratch);
+    if (kind == NORM_LAYER) ss = centre_row(row, H, sum, scratch);
+    else ss = block_sum(ss, scratch);
     const float inv = 1.f / sqrtf(ss / (float)H + eps);
     for (int c = threadIdx.x; c < H; c += R32_THREADS) nr[c] = from_f32<T>((row[c] * inv) * w[c]);
 }
@@ -190,20 +170,6 @@ extern "C" int cm_norm_f32in(int dt, void* y, const float* x, const float* w, in
         return CM_ERR_DTYPE;
     CM_CHECK_LAUNCH();
     return CM_OK;
-}
-
-static void fill_terms(ResidualTerms& terms, int n_terms, const void* const* term_ptr, const float* term_scale,
-                       const int* term_per_row, const int* term_is_f32, const int* const* term_index,
-                       const float* const* term_weights) {
-    terms.n = n_terms;
-    for (int i = 0; i < R32_MAX_TERMS; ++i) {
-        terms.t[i].p = i < n_terms ? term_ptr[i] : nullptr;
-        terms.t[i].index = i < n_terms ? term_index[i] : nullptr;
-        terms.t[i].weights = i < n_terms ? term_weights[i] : nullptr;
-        terms.t[i].scale = i < n_terms ? term_scale[i] : 0.f;
-        terms.t[i].per_row = i < n_terms ? term_per_row[i] : 0;
-        terms.t[i].is_f32 = i < n_terms ? term_is_f32[i] : 0;
-    }
 }
 
 // terms: n_terms entries of (pointer, scale, pieces per row, stored as float?, index of the pieces or null, a weight per

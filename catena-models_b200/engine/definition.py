@@ -48,6 +48,9 @@ class ModelDefinition:
     residual_float32: bool = False   # the residual stream is float32 whatever the activation dtype (the blocks must take it)
     keep_embedding: bool = False     # a copy of the embedding rows stays in StepBatch.shared["embedding"] for the blocks
     embedding_norm: object = None    # an RMS norm over every embedding row (a float32 stream), before the first block
+    # > 0: the residual is this many hyper-connected streams, float32 [rows, streams, width]: the first block's input norm (a
+    # `streams` norm) opens them from the embedding rows, the final norm reads their sum
+    streams: int = 0
     # > 0: blocks average over the depth of the stack; the step keeps the stream before the first block and after every
     # block in StepBatch.shared["depth_history"] (float32 [depth_entries, rows, width]); the model fills entry 0
     depth_entries: int = 0

@@ -131,7 +131,9 @@ class DecoderModel:
         d = self.definition
         if d.embedding_norm is not None or d.depth_entries:
             n = self._prepare_stream(rt, batch, h, first_norm is None)
-        if first_norm is not None:
+        if d.streams:
+            h, n = first_norm.open(rt, h)
+        elif first_norm is not None:
             n = first_norm.apply(rt, h)
         # when every row is wanted in order (a decode step), the last block's fused residual kernel
         # applies the final norm too and no rows need gathering
@@ -153,8 +155,8 @@ class DecoderModel:
         if whole and n is not None:
             logits = rt.linear(n, self.head_weight, out_dtype=torch.float32)
         else:
-            rows = torch.empty((batch.n_want, self.hidden_size), dtype=h.dtype, device=rt.device)
-            kernels.gather_rows(rows, h, batch.want_rows)
+            rows = torch.empty((batch.n_want, *h.shape[1:]), dtype=h.dtype, device=rt.device)
+            kernels.gather_rows(rows.view(batch.n_want, -1), h.view(batch.T, -1), batch.want_rows)
             normed = self.final_norm.apply(rt, rows)
             logits = rt.linear(normed, self.head_weight, out_dtype=torch.float32)
         if d.logit_scale != 1.0 or d.logit_softcap > 0.0:

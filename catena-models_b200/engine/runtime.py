@@ -306,7 +306,7 @@ class Runtime:
         aligned = (q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and k.data_ptr() % 16 == 0
                    and v.data_ptr() % 16 == 0)
         bf16 = q.dtype == torch.bfloat16 and self.tensor_core_prompts
-        span = min(batch.max_len, window) if window else batch.max_len
+        span = min(batch.max_len, abs(window)) if window else batch.max_len
         long_enough = span >= self.TCGEN05_ATTENTION_MIN_LEN or (
             span >= self.TCGEN05_ATTENTION_MIN_LEN_BATCH and q.shape[0] >= self.TCGEN05_ATTENTION_MIN_TOKENS)
         if (bf16 and aligned and HD in (64, 128) and long_enough
@@ -334,7 +334,7 @@ class Runtime:
         aligned = (q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and k.data_ptr() % 16 == 0
                    and v.data_ptr() % 16 == 0 and state.pool.data_ptr() % 16 == 0)
         bf16 = q.dtype == torch.bfloat16 and state.pool.dtype == torch.bfloat16 and self.tensor_core_prompts
-        span = min(batch.max_end, window) if window else batch.max_end
+        span = min(batch.max_end, abs(window)) if window else batch.max_end
         if (bf16 and aligned and HD in (64, 128) and span >= self.TCGEN05_APPEND_MIN_SPAN
                 and batch.max_len >= self.TCGEN05_APPEND_MIN_ROWS and ctx.stride(0) % 8 == 0 and ctx.data_ptr() % 16 == 0):
             kernels.attn_append_tc(ctx, q, k, v, gate, batch.seq_start, batch.seq_pos0, batch.seq_slot, state.pool,

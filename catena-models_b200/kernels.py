@@ -33,7 +33,7 @@ _SIGNATURES = {
     "cm_gemm_tc": [_i, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _f, _vp],
     "cm_gemm_tc_few_rows": [_i, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _f, _vp],
     "cm_qk_prepare": [_i, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _i,
-                      _i, _f, _i, _f, _i, _vp],
+                      _i, _i, _f, _i, _f, _i, _vp],
     "cm_attn_prefill_simt": [_i, _vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp],
     "cm_attn_prefill_mma": [_vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp],
     "cm_attn_prefill_tc": [_vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _ll, _i, _i, _i, _i, _f, _f, _vp, _vp, _vp],
@@ -56,6 +56,9 @@ _SIGNATURES = {
     "cm_norm_f32in": [_i, _vp, _vp, _vp, _i, _i, _f, _i, _vp, _vp, _vp],
     "cm_residual_add_norm": [_i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp, _vp, _vp],
     "cm_postnorm_residual": [_i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _f, _vp, _i, _i, _f, _vp, _ll, _i, _vp, _vp],
+    "cm_hyper_connect": [_i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _f, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "cm_delta_prompt": [_i, _vp, _vp],
+    "cm_delta_step": [_i, _vp, _vp],
     "cm_relu2_inplace": [_i, _vp, _ll, _vp],
     "cm_tap_rotate_store": [_i, _vp, _vp],
     "cm_diff_attn": [_i, _vp, _i, _i, _vp, _i, _vp],
@@ -68,7 +71,7 @@ _SIGNATURES = {
     "cm_decay_from_logits": [_vp, _vp, _vp, _ll, _i, _i, _f, _vp],
     "cm_matrix_scan": [_i, _i, _vp, _i, _vp],
     "cm_lightning_chunked": [_i, _vp, _i, _i, _vp, _vp],
-    "cm_moe_route": [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _i, _i, _i, _f, _f, _i, _vp],
+    "cm_moe_route": [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _i, _i, _i, _f, _f, _i, _vp, _vp],
     "cm_moe_identity": [_i, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _vp],
     "cm_latent_prepare": [_i, _vp, _vp],
     "cm_latent_query_turn": [_i, _vp, _vp],
@@ -562,16 +565,17 @@ def gemm_tc_few_rows(y, x, w, swiglu=False, err=None, splits=0, limit=0.0):
 
 # -------------------------------------------------------------------------- attention
 def qk_prepare(qkv, wq, wk, rate, tok_pos, tok_seq, seq_slot, seq_end, pool, pages, ptab, ring,
-               QH, KVH, HD, eps, interleaved=False, q_temp=None):
+               QH, KVH, HD, eps, interleaved=False, q_temp=None, norm_dim=None):
     """Head norm + rotation in place on the q and k columns of qkv; k and v go to the cache
     (pool: this layer's [2, pages, KVH, 64, HD] storage, or None to write no cache).  The rotation
     pairs element i with i + HD/2, or, with `interleaved`, 2i with 2i + 1.  `q_temp` = (coef, every):
-    the queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)."""
+    the queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).  `norm_dim`: the channels that
+    the head norm's mean of squares counts, when the others of a head are zero padding."""
     qt_coef, qt_every = (float(q_temp[0]), int(q_temp[1])) if q_temp else (0.0, 0)
     T = qkv.shape[0]
     _check(lib().cm_qk_prepare(dtype_code(qkv.dtype), _ptr(qkv), qkv.stride(0), _ptr(wq), _ptr(wk), _ptr(rate),
                                _ptr(tok_pos), _ptr(tok_seq), _ptr(seq_slot), _ptr(seq_end), _ptr(pool), pages,
-                               _ptr(ptab), 0 if ptab is None else ptab.stride(0), ring, T, QH, KVH, HD, eps,
+                               _ptr(ptab), 0 if ptab is None else ptab.stride(0), ring, T, QH, KVH, HD, norm_dim or HD, eps,
                                int(interleaved), qt_coef, qt_every, _stream()), "qk_prepare",
            cost=lambda: (f"{T} tokens, {QH}+{KVH} heads of {HD}",
                          T * HD * qkv.element_size() * (2 * QH + (2 * KVH if pool is None else 4 * KVH)), 0))
@@ -581,7 +585,9 @@ def attn_prefill_simt(ctx, q, k, v, gate, seq_start, B, max_len, QH, KVH, HD, wi
     """q, k, v, gate are column views of one packed row-major buffer (same row stride).  `sink` (all
     attention kernels): float32 [QH], a learned logit per query head that joins the softmax's denominator
     and nothing else (it has no key and no value), or None.  `softcap` (all attention kernels) = c > 0: every
-    score is bounded before the mask and the softmax, s <- c * tanh(s / c) with s = (q . k) * scale."""
+    score is bounded before the mask and the softmax, s <- c * tanh(s / c) with s = (q . k) * scale.  `window` (all
+    attention kernels): W > 0, a query sees the last W positions; W < 0, the positions of its own chunk, chunks of -W
+    positions counted from the sequence's start; 0, every earlier position."""
     if not (q.stride(0) == k.stride(0) == v.stride(0)):
         raise KernelError("attn_prefill: q, k and v must share a row stride")
     _check(lib().cm_attn_prefill_simt(dtype_code(q.dtype), _ptr(ctx), ctx.stride(0), _ptr(q), _ptr(k), _ptr(v),
@@ -764,17 +770,18 @@ def zero_slots(store, slots):
 
 
 # ------------------------------------------------------------------ float residual stream
-NORM_RMS, NORM_DYT = 0, 1          # csrc/residual32.cu
+NORM_RMS, NORM_DYT, NORM_LAYER = 0, 1, 2          # csrc/residual32.cu
 
 
-def norm_f32in(out, x, w, eps, dyt=None):
+def norm_f32in(out, x, w, eps, dyt=None, layer=False):
     """out = norm(x) * w for float32 rows x; out in the activation dtype.  `dyt` = (alpha, shift): a dynamic
-    tanh instead, out = tanh(alpha x) * w + shift (alpha a float32 tensor of one element, shift float32 [H])."""
+    tanh instead, out = tanh(alpha x) * w + shift (alpha a float32 tensor of one element, shift float32 [H]).
+    `layer`: a layer norm without a shift instead of a root-mean-square norm."""
     _need_cuda(out, x, w)
     rows, H = x.shape
     if x.dtype != torch.float32 or not x.is_contiguous() or not out.is_contiguous():
         raise KernelError("norm_f32in takes contiguous float32 rows")
-    kind, alpha, shift = (NORM_DYT, dyt[0], dyt[1]) if dyt is not None else (NORM_RMS, None, None)
+    kind, alpha, shift = (NORM_DYT, dyt[0], dyt[1]) if dyt is not None else (NORM_LAYER if layer else NORM_RMS, None, None)
     _check(lib().cm_norm_f32in(dtype_code(out.dtype), _ptr(out), _ptr(x), _ptr(w), rows, H, eps, kind, _ptr(alpha),
                                _ptr(shift), _stream()), "norm_f32in",
            cost=lambda: (f"{rows}x{H}", _nbytes(x, out, w), 4 * rows * H))
@@ -809,16 +816,16 @@ def _term_arrays(terms, rows, H, act, name):
     return terms, n, ptrs, scales, per, f32, index, weights
 
 
-def residual_add_norm(h, terms, n_out=None, w_next=None, eps=0.0, bias=None, dyt=None):
+def residual_add_norm(h, terms, n_out=None, w_next=None, eps=0.0, bias=None, dyt=None, layer=False):
     """h (float32, in place) += sum over `terms` of scale * (the sum of a row's pieces) (+ bias, a float32
     row); n_out = norm(h) * w_next in the activation dtype when given (`dyt` = (alpha, shift): a dynamic tanh,
-    as for `norm_f32in`).  A term is (tensor, scale, pieces per row[, index[, weights]]): see `Terms`."""
+    as for `norm_f32in`; `layer`: a layer norm).  A term is (tensor, scale, pieces per row[, index[, weights]]): see `Terms`."""
     rows, H = h.shape
     if h.dtype != torch.float32 or not h.is_contiguous():
         raise KernelError("residual_add_norm: a contiguous float32 stream")
     act = n_out.dtype if n_out is not None else next((t[0].dtype for t in terms if t[0].dtype != torch.float32), torch.float32)
     terms, n, ptrs, scales, per, f32, index, weights = _term_arrays(terms, rows, H, act, "residual_add_norm")
-    kind, alpha, shift = (NORM_DYT, dyt[0], dyt[1]) if dyt is not None else (NORM_RMS, None, None)
+    kind, alpha, shift = (NORM_DYT, dyt[0], dyt[1]) if dyt is not None else (NORM_LAYER if layer else NORM_RMS, None, None)
     _check(lib().cm_residual_add_norm(dtype_code(act), _ptr(h), _ptr(n_out), n, ptrs, scales, per, f32, index, weights, _ptr(bias),
                                       _ptr(w_next), rows, H, eps, kind, _ptr(alpha), _ptr(shift), _stream()), "residual_add_norm",
            cost=lambda: (f"{rows}x{H}, {n} terms", 2 * _nbytes(h) + _nbytes(n_out) + sum(rows * t[2] * H * t[0].element_size() for t in terms),
@@ -846,6 +853,36 @@ def postnorm_residual(h, terms, h_scale, w, eps, n_out=None, history=None, coef=
            "postnorm_residual",
            cost=lambda: (f"{rows}x{H}, {n} terms, depth {n_hist}", 2 * _nbytes(h) + _nbytes(n_out) + (n_hist + 1) * rows * H * 4
                          + sum(rows * t[2] * H * t[0].element_size() for t in terms), (n + 5 + 2 * n_hist) * rows * H))
+
+
+HYPER_MAX_STREAMS = 8              # csrc/hyper.cu: HC_MAX_STREAMS
+
+
+def hyper_connect(x, terms=(), mix=None, put=None, n_out=None, read=None, w=None, eps=0.0, out=None):
+    """Hyper-connected streams, float32 [rows, S, W].  With `mix` [S, S] and `put` [S]: the write behind a sublayer whose
+    result is the sum of `terms` (as for `residual_add_norm`), X_t <- sum_s mix[s, t] X_s + put[t] y, in place of x.  With
+    `n_out` (activation dtype, [rows, W]): the read in front of the next sublayer, the layer norm (weight w) of sum_s
+    read[s] X_s.  x of two dimensions [rows, W] with `out` [rows, S, W] opens the streams: every one becomes x.  Without
+    `mix` and `out` the streams stay as they are.  mix, put, read, w: float32 on the device."""
+    open_, streams = x.dim() == 2, out if x.dim() == 2 else x
+    rows, S, W = streams.shape
+    for t in (x, streams):
+        if t.dtype != torch.float32 or not t.is_contiguous():
+            raise KernelError("hyper_connect: contiguous float32 streams")
+    if open_ and (tuple(x.shape) != (rows, W) or mix is not None):
+        raise KernelError("hyper_connect: opening takes rows [rows, W] and mixes nothing")
+    for t, n in ((mix, S * S), (put, S), (read, S), (w, W)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous()):
+            raise KernelError("hyper_connect: a constant's size or dtype does not fit")
+    if n_out is not None and (tuple(n_out.shape) != (rows, W) or not n_out.is_contiguous()):
+        raise KernelError("hyper_connect: the normed rows are [rows, W]")
+    act = n_out.dtype if n_out is not None else next((t[0].dtype for t in terms if t[0].dtype != torch.float32), torch.float32)
+    terms, n, ptrs, scales, per, f32, index, weights = _term_arrays(terms, rows, W, act, "hyper_connect")
+    write = streams if open_ or mix is not None else None
+    _check(lib().cm_hyper_connect(dtype_code(act), _ptr(write), _ptr(x), int(open_), _ptr(mix), _ptr(put), _ptr(read), _ptr(w), eps,
+                                  _ptr(n_out), n, ptrs, scales, per, f32, index, weights, rows, S, W, _stream()), "hyper_connect",
+           cost=lambda: (f"{rows}x{S}x{W}, {n} terms", _nbytes(x, write, n_out) + sum(rows * t[2] * W * t[0].element_size() for t in terms),
+                         rows * W * (2 * S * S + 2 * S + 8)))
 
 
 def concat_cast(out, a, b):
@@ -952,6 +989,69 @@ def matrix_scan(mode, out, q, k, v, g, decay, bonus, norm_w, state, state_offset
            cost=lambda: (f"{B} sequences, {rows} rows, {H} heads of {D}x{DV}",
                          _nbytes(q, k, v, g, out) + (0 if decay is None or decay.dim() < 2 else rows * decay.shape[1] * 4) + 2 * B * H * D * DV * 4,
                          6 * rows * H * D * DV))
+
+
+class _DeltaArgs(ctypes.Structure):
+    """csrc/delta.h: DeltaArgs."""
+    _fields_ = [("proj", _vp), ("ldp", _ll), ("gates", _vp), ("ldg", _ll), ("x", _vp), ("w_gates", _vp), ("W", _i), ("rate", _vp),
+                ("dt_bias", _vp), ("taps", _vp), ("norm_w", _vp), ("state", _vp), ("state_stride", _ll), ("out", _vp), ("ldo", _ll),
+                ("qk", _vp), ("v", _vp), ("lb", _vp), ("raw", _vp), ("tok_seq", _vp), ("tok_pos", _vp), ("seq_start", _vp),
+                ("seq_pos0", _vp), ("seq_slot", _vp), ("rows", _ll), ("B", _i), ("H", _i), ("G", _i), ("D", _i), ("DV", _i), ("K", _i),
+                ("q_scale", _f), ("unit_eps", _f), ("eps", _f), ("from_zero", _i), ("chunks", _vp), ("max_len", _i)]
+
+
+def delta_step_fits(D, DV):
+    """True if `delta_rule` can run a step of single tokens as one kernel for heads of D x DV."""
+    fn = lib().cm_delta_step_fits
+    fn.argtypes, fn.restype = [_i, _i], _i
+    return bool(fn(D, DV))
+
+
+def delta_state_floats(H, G, D, DV, K):
+    """Floats of a sequence's state row: S [H, D, DV], then a ring of K projected rows (none for K = 1), rounded up to
+    whole 16-byte pieces."""
+    return -(-(H * D * DV + (K * (2 * G * D + H * DV) if K > 1 else 0)) // 4) * 4
+
+
+def delta_rule(out, proj, taps, rate, dt_bias, norm_w, state, batch, H, G, D, DV, q_scale, unit_eps, eps, gates=None, x=None,
+               w_gates=None):
+    """The gated delta rule behind its projections (csrc/delta.cu).  proj [rows, n]: q (G D channels) | k (G D) | v (H DV) |
+    output gate (H DV), activation dtype; taps float32 [2 G D + H DV, K]; rate, dt_bias float32 [H]; norm_w float32 [H DV];
+    state float32 [slots, delta_state_floats]; out [rows, H DV].  `gates` float32 [rows, >= 2 H]: the pre-activations of
+    beta, then of the decay, for a step of any lengths; or, for a step of one token per sequence whose heads fit
+    (`delta_step_fits`), the mixer's input `x` [rows, W] and the gate projections' rows `w_gates` [2 H, W]: one kernel."""
+    rows, C, K = proj.shape[0], 2 * G * D + H * DV, taps.shape[1]
+    if taps.shape[0] != C or proj.shape[1] < C + H * DV or proj.stride(1) != 1 or out.dtype != proj.dtype or out.stride(1) != 1:
+        raise KernelError("delta_rule: the projected rows do not hold the channels that the taps name")
+    for t, n in ((taps, C * K), (rate, H), (dt_bias, H), (norm_w, H * DV)):
+        if t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous():
+            raise KernelError("delta_rule: a constant's size or dtype does not fit")
+    if state.dtype != torch.float32 or state.shape[-1] < delta_state_floats(H, G, D, DV, K):
+        raise KernelError("delta_rule: a float32 state row per slot")
+    a = _DeltaArgs(proj=_ptr(proj), ldp=proj.stride(0), rate=_ptr(rate), dt_bias=_ptr(dt_bias), taps=_ptr(taps), norm_w=_ptr(norm_w),
+                   state=_ptr(state), state_stride=state.stride(0), out=_ptr(out), ldo=out.stride(0), tok_seq=_ptr(batch.tok_seq),
+                   tok_pos=_ptr(batch.tok_pos), seq_start=_ptr(batch.seq_start), seq_pos0=_ptr(batch.seq_pos0),
+                   seq_slot=_ptr(batch.seq_slot), rows=rows, B=batch.B, H=H, G=G, D=D, DV=DV, K=K, q_scale=q_scale,
+                   unit_eps=unit_eps, eps=eps, from_zero=int(batch.kind == "prefill"), max_len=batch.max_len)
+    flops = 8 * rows * H * D * DV
+    moved = _nbytes(proj, out) + 2 * batch.B * H * D * DV * 4
+    if gates is None:
+        if batch.kind != "decode" or x.dtype != proj.dtype or w_gates.dtype != proj.dtype or not (x.is_contiguous() and w_gates.is_contiguous()):
+            raise KernelError("delta_rule: the one-kernel form is for steps of single tokens, operands of one dtype")
+        a.x, a.w_gates, a.W = _ptr(x), _ptr(w_gates), x.shape[1]
+        _check(lib().cm_delta_step(dtype_code(proj.dtype), ctypes.byref(a), _stream()), "delta_step",
+               cost=lambda: (f"{rows} sequences, {H}/{G} heads of {D}x{DV}, {K} taps", moved, flops))
+        return
+    if gates.dtype != torch.float32 or gates.shape[0] != rows or gates.shape[1] < 2 * H:
+        raise KernelError("delta_rule: float32 gate pre-activations [rows, 2 H]")
+    qk = torch.empty((rows, 2 * G * D), dtype=torch.float32, device=proj.device)
+    v = torch.empty((rows, H * DV), dtype=proj.dtype, device=proj.device)
+    lb = torch.empty((rows, 2 * H), dtype=torch.float32, device=proj.device)
+    raw = torch.empty((rows, H * DV), dtype=torch.float32, device=proj.device)
+    a.gates, a.ldg, a.qk, a.v, a.lb, a.raw = _ptr(gates), gates.stride(0), _ptr(qk), _ptr(v), _ptr(lb), _ptr(raw)
+    _check(lib().cm_delta_prompt(dtype_code(proj.dtype), ctypes.byref(a), _stream()), "delta_prompt",
+           3 if K < 2 or a.from_zero else 4,
+           cost=lambda: (f"{batch.B} sequences, {rows} rows, {H}/{G} heads of {D}x{DV}, {K} taps", moved, flops))
 
 
 LIGHTNING_CHUNK = 64               # csrc/lightning.cu: rows of a chunk of the prompt form
@@ -1259,10 +1359,14 @@ def moe_tile_group(work, pairs, experts, tile_rows):
     return work[2 * experts + 1 + 3 * tiles:2 * experts + 1 + 4 * tiles]
 
 
+MOE_GATES = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}       # csrc/moe.cu: RouteRule.gate
+
+
 def moe_route(ids, wts, perm, dest, work, h, w_router, tok_seq, top, softmax_gate=False, renormalize=False,
               tile_rows=MOE_TILE_SIMT, xs=None, apply_weight=False, correction=None, groups=0, keep=0, identity=0, scale=1.0,
-              renorm_eps=0.0, group_best=1):
-    """Scores of every token's experts in float32 (sigmoid, or softmax over the experts), the `top` best
+              renorm_eps=0.0, group_best=1, gate=None, bias=None):
+    """Scores of every token's experts in float32 (`gate`: "sigmoid", "softmax" over the experts, or "softmax_chosen": the
+    logits themselves, with a softmax over the chosen ones as weights; `bias`, float32 [E], is added to the logits), the `top` best
     (ids, wts: [rows * top]; -1 for rows of padding), and the pairs in the order of their experts, every expert's
     rows beginning a row tile of `tile_rows` rows: perm[sorted row] = pair (moe_max_tiles * tile_rows entries),
     dest[pair] = sorted row (-1: none), the list of row tiles in `work` (int32, moe_work_size entries).  With `xs`
@@ -1276,14 +1380,17 @@ def moe_route(ids, wts, perm, dest, work, h, w_router, tok_seq, top, softmax_gat
     `renormalize` divides by."""
     rows, W = h.shape
     E = w_router.shape[0]
+    gate = MOE_GATES[gate] if gate is not None else int(bool(softmax_gate))
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != E):
+        raise KernelError("moe_route: one float32 bias per router output")
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E):
         raise KernelError("moe_route: one float32 correction per router output")
     if w_router.dtype != h.dtype or not (h.is_contiguous() and w_router.is_contiguous()):
         raise KernelError("moe_route: contiguous operands of one dtype")
     _check(lib().cm_moe_route(dtype_code(h.dtype), _ptr(ids), _ptr(wts), _ptr(perm), _ptr(dest), _ptr(work), _ptr(h),
-                              _ptr(w_router), _ptr(tok_seq), rows, W, E, top, int(softmax_gate), int(renormalize), tile_rows,
+                              _ptr(w_router), _ptr(tok_seq), rows, W, E, top, gate, int(renormalize), tile_rows,
                               _ptr(xs), int(apply_weight), _ptr(correction), int(groups), int(keep), int(identity), float(scale),
-                              float(renorm_eps), int(group_best), _stream()), "moe_route",
+                              float(renorm_eps), int(group_best), _ptr(bias), _stream()), "moe_route",
            1 if rows <= 64 and rows * E * (2 if correction is not None or groups else 1) <= 8192 else (4 if xs is not None else 3),
            cost=lambda: (f"{rows}x{W} over {E}, top {top}", _nbytes(h, w_router), 2 * rows * E * W))
 

@@ -23,6 +23,10 @@ and the cache work with one head size, so heads of unequal or odd sizes are padd
 projections up to a common multiple of 16 (zero channels change no score and give zero outputs, which meet
 zero columns of the output projection); `out_dtype` = "float32" leaves the output projection's result in float.
 
+`chunk` = C > 0 (instead of a window): position p sees the earlier positions of its own chunk of C, chunks counted from the
+sequence's start; the cache is a ring that holds the last C positions, as for a window of C.  `sink_value`: a constant logit
+for every query head in place of the learned ones.  With a head norm, padded heads are normed over their real channels.
+
 `softcap` = c > 0 bounds every score before the mask and the softmax: s <- c * tanh(s / c), s = (q . k) * scale.
 
 `taps` = K >= 1 puts a short causal filter behind the query and key projections, one set of K taps per channel
@@ -52,14 +56,12 @@ class GQAttention(Mixer):
 
     def __init__(self, prefix, hidden, heads, kv_heads, head_dim, window, position, qk_norm_eps,
                  output_gate, names=None, shares_kv=False, scale=None, sink_name=None, q_temp=None, value_dim=None,
-                 out_dtype=None, softcap=0.0, taps=0, value_from_key=False):
+                 out_dtype=None, softcap=0.0, taps=0, value_from_key=False, chunk=0, sink_value=None):
         names = names or {}
         n = lambda key, default: prefix + names.get(key, default)
         qk_dim, v_dim = head_dim, value_dim or head_dim
         if v_dim != qk_dim or (scale is not None and qk_dim % 16):
             head_dim = -(-max(qk_dim, v_dim) // 16) * 16       # one padded head size for q, k and v
-            if qk_norm_eps is not None and head_dim != qk_dim:
-                raise ValueError("a head norm over padded heads is not built")
         pad_qk = (heads, qk_dim, head_dim) if head_dim != qk_dim else None
         pad_k = (kv_heads, qk_dim, head_dim) if head_dim != qk_dim else None
         pad_v = (kv_heads, v_dim, head_dim) if head_dim != v_dim else None
@@ -78,7 +80,14 @@ class GQAttention(Mixer):
         self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp else None
         self.out_dtype = {None: None, "float32": torch.float32}[out_dtype]
         self.hidden, self.heads, self.kv_heads, self.head_dim = hidden, heads, kv_heads, head_dim
+        if chunk and window:
+            raise ValueError("GQAttention: a window or chunks, not both")
+        if sink_name and sink_value is not None:
+            raise ValueError("GQAttention: learned sinks or a constant one")
+        self.sink_value = sink_value
         self.window = int(window or 0)
+        self.reach = self.window or int(chunk or 0)          # how many positions the cache keeps (0: all)
+        self.mask = -int(chunk) if chunk else self.window    # the mask as the attention kernels take it
         self.position = position
         self.qk_norm_eps = qk_norm_eps           # None: no head norm
         self.output_gate = bool(output_gate)
@@ -121,9 +130,9 @@ class GQAttention(Mixer):
                       TensorSpec(self.tap_names[1], (self.kv_heads * self.qk_dim, self.taps), "conv")]
         if self.qk_norm_eps is None:
             return specs
-        specs.append(TensorSpec(self.q_norm_name, (self.head_dim,), "norm"))
+        specs.append(TensorSpec(self.q_norm_name, (self.qk_dim,), "norm"))
         if not self.shares_kv:
-            specs.append(TensorSpec(self.k_norm_name, (self.head_dim,), "norm"))
+            specs.append(TensorSpec(self.k_norm_name, (self.qk_dim,), "norm"))
         return specs
 
     def bind(self, tensors, rt):
@@ -144,15 +153,19 @@ class GQAttention(Mixer):
         if self.sink_name:
             self.sink = tensors[self.sink_name].to(torch.float32).contiguous()
             self._bound.append(self.sink)
+        elif self.sink_value is not None:
+            self.sink = torch.full((self.heads,), float(self.sink_value), dtype=torch.float32, device=rt.device)
+            self._bound.append(self.sink)
         if self.qk_norm_eps is not None:
-            self.q_norm_w = tensors[self.q_norm_name].to(torch.float32).contiguous()
+            padded = lambda w: torch.nn.functional.pad(w.to(torch.float32), (0, self.head_dim - self.qk_dim)).contiguous()
+            self.q_norm_w = padded(tensors[self.q_norm_name])
             self._bound.append(self.q_norm_w)
             if not self.shares_kv:
-                self.k_norm_w = tensors[self.k_norm_name].to(torch.float32).contiguous()
+                self.k_norm_w = padded(tensors[self.k_norm_name])
                 self._bound.append(self.k_norm_w)
 
     def state_spec(self):
-        kv = KVStateSpec(self.kv_heads, self.head_dim, self.window)
+        kv = KVStateSpec(self.kv_heads, self.head_dim, self.reach)
         if self.taps > 1:
             # a ring of `taps` projected rows [q | k] per sequence, the row of position s in row s % taps
             return CompositeStateSpec((kv, FixedStateSpec((self.taps * (self.q_size + self.kv_size),), "float32")))
@@ -180,17 +193,17 @@ class GQAttention(Mixer):
             n_chunks = max(1, -(-entries // ATTN_DECODE_CHUNK))
             part_o, part_ml = rt.scratch_attn_decode(batch.B, QH, HD, n_chunks)
             kernels.attn_decode(ctx, q, None, batch.seq_pos0, batch.seq_slot, kv.pool, kv.pages, kv.ptab, kv.ring,
-                                self.window, QH, KVH, HD, n_chunks, self.scale, part_o, part_ml, sink=self.sink,
+                                self.mask, QH, KVH, HD, n_chunks, self.scale, part_o, part_ml, sink=self.sink,
                                 softcap=self.softcap)
         else:
             k, v = packed[:, QS:QS + KVS], packed[:, QS + KVS:]
             if batch.append:
-                rt.attention_append(ctx, q, k, v, None, batch, kv, QH, KVH, HD, self.window, self.scale, sink=self.sink,
+                rt.attention_append(ctx, q, k, v, None, batch, kv, QH, KVH, HD, self.mask, self.scale, sink=self.sink,
                                     softcap=self.softcap)
                 kernels.kv_store(packed[:, QS:], batch.tok_pos, batch.tok_seq, batch.seq_slot, batch.seq_end, kv.pool,
                                  kv.pages, kv.ptab, kv.ring, KVH, HD)
             else:
-                rt.attention_prefill(ctx, q, k, v, None, batch, QH, KVH, HD, self.window, self.scale, sink=self.sink,
+                rt.attention_prefill(ctx, q, k, v, None, batch, QH, KVH, HD, self.mask, self.scale, sink=self.sink,
                                      softcap=self.softcap)
         return self.out.apply(rt, ctx, out_dtype=self.out_dtype)
 
@@ -207,14 +220,15 @@ class GQAttention(Mixer):
             # q only: head norm and rotation over the q heads, nothing written to the cache
             kernels.qk_prepare(proj, self.q_norm_w, None, self.position.rate_table(), batch.tok_pos, batch.tok_seq,
                                batch.seq_slot, batch.seq_end, None, 0, None, 0, QH, 0, HD, self.qk_norm_eps or 0.0,
-                               interleaved=interleaved, q_temp=self.q_temp)
+                               interleaved=interleaved, q_temp=self.q_temp, norm_dim=self.qk_dim)
             gate = proj[:, QS:] if self.output_gate else None
         else:
             # an append step keeps the cache as it is until its attention has run
             pool = None if batch.append else state.pool
             kernels.qk_prepare(proj, self.q_norm_w, self.k_norm_w, self.position.rate_table(), batch.tok_pos,
                                batch.tok_seq, batch.seq_slot, batch.seq_end, pool, state.pages, state.ptab,
-                               state.ring, QH, KVH, HD, self.qk_norm_eps or 0.0, interleaved=interleaved, q_temp=self.q_temp)
+                               state.ring, QH, KVH, HD, self.qk_norm_eps or 0.0, interleaved=interleaved, q_temp=self.q_temp,
+                               norm_dim=self.qk_dim)
             gate = proj[:, QS + 2 * KVS:] if self.output_gate else None
         q = proj[:, :QS]
         ctx = torch.empty((batch.T, QS), dtype=x.dtype, device=x.device)
@@ -235,13 +249,13 @@ class GQAttention(Mixer):
                 k, v = proj[:, QS:QS + KVS], proj[:, QS + KVS:QS + 2 * KVS]
                 batch.shared[("kv", state.unit)] = (k, v)
             if batch.append:
-                rt.attention_append(ctx, q, k, v, gate, batch, state, QH, KVH, HD, self.window, self.scale, sink=self.sink,
+                rt.attention_append(ctx, q, k, v, gate, batch, state, QH, KVH, HD, self.mask, self.scale, sink=self.sink,
                                     softcap=self.softcap)
                 if not self.shares_kv:
                     kernels.kv_store(proj[:, QS:QS + 2 * KVS], batch.tok_pos, batch.tok_seq, batch.seq_slot,
                                      batch.seq_end, state.pool, state.pages, state.ptab, state.ring, KVH, HD)
             else:
-                rt.attention_prefill(ctx, q, k, v, gate, batch, QH, KVH, HD, self.window, self.scale, sink=self.sink,
+                rt.attention_prefill(ctx, q, k, v, gate, batch, QH, KVH, HD, self.mask, self.scale, sink=self.sink,
                                      softcap=self.softcap)
         else:
             # launched for the longest sequence that this step's length class allows, so that a
@@ -250,7 +264,7 @@ class GQAttention(Mixer):
             n_chunks = max(1, -(-entries // ATTN_DECODE_CHUNK))
             part_o, part_ml = rt.scratch_attn_decode(batch.B, QH, HD, n_chunks)
             kernels.attn_decode(ctx, q, gate, batch.seq_pos0, batch.seq_slot, state.pool, state.pages, state.ptab,
-                                state.ring, self.window, QH, KVH, HD, n_chunks, self.scale, part_o, part_ml, sink=self.sink,
+                                state.ring, self.mask, QH, KVH, HD, n_chunks, self.scale, part_o, part_ml, sink=self.sink,
                                 softcap=self.softcap)
         return self.out.apply(rt, ctx, out_dtype=self.out_dtype, partial_ok=batch.partial_sums_ok and self.out_dtype is None)
 

@@ -19,6 +19,9 @@ times the weight; they take part in scores, groups and choice like any other); `
 `renorm_eps` (added to the sum that `renormalize` divides by); `group_best` (a group's score is the sum of that many of its
 largest choice scores instead of the largest alone).
 
+`gate` "softmax_chosen": the scores are the logits themselves and the weights a softmax over the chosen experts' logits
+alone; `bias_name`: a tensor of one number per router output, added to the logits (it counts in the choice and in the weights).
+
 `activation` "clamped_swish" with `limit` L is an expert of another form: g = min(W_gate x, L), u = clamp(W_up x, -L, L),
 a = g sigmoid(1.702 g) (u + 1).
 """
@@ -37,16 +40,17 @@ class RoutedSwiGLU(FeedForward):
 
     def __init__(self, prefix, hidden, intermediate, experts, top, gate="sigmoid", renormalize=False,
                  weight_on="input", activation="silu", expert_name="e{}.", correction_name=None, groups=0, keep=0,
-                 identity=0, scale=1.0, renorm_eps=0.0, group_best=1, limit=0.0):
-        if gate not in ("sigmoid", "softmax") or weight_on not in ("input", "output") or activation not in kernels.ACTIVATIONS:
-            raise ValueError("RoutedSwiGLU: gate sigmoid|softmax, weight_on input|output, activation silu|gelu_tanh|clamped_swish")
+                 identity=0, scale=1.0, renorm_eps=0.0, group_best=1, limit=0.0, bias_name=None):
+        if gate not in kernels.MOE_GATES or weight_on not in ("input", "output") or activation not in kernels.ACTIVATIONS:
+            raise ValueError("RoutedSwiGLU: gate sigmoid|softmax|softmax_chosen, weight_on input|output, activation silu|gelu_tanh|clamped_swish")
         if activation == "clamped_swish" and not limit > 0.0:
             raise ValueError("RoutedSwiGLU: the clamped gate needs its limit")
         if top < 1 or experts < 1:
             raise ValueError(f"RoutedSwiGLU: {top} of {experts} experts")
         self.prefix, self.hidden, self.intermediate = prefix, hidden, intermediate
         self.experts, self.top = experts, top
-        self.softmax_gate, self.renormalize = gate == "softmax", bool(renormalize)
+        self.gate, self.renormalize = gate, bool(renormalize)
+        self.bias_name, self.bias = bias_name, None
         self.weight_on_input, self.gelu = weight_on == "input", activation == "gelu_tanh"
         self.act, self.limit, self.group_best = kernels.ACTIVATIONS[activation], float(limit), int(group_best or 1)
         self.expert_name = expert_name
@@ -71,6 +75,8 @@ class RoutedSwiGLU(FeedForward):
         specs = [TensorSpec(self.prefix + "router", (self.outputs, H))]
         if self.correction_name:
             specs.append(TensorSpec(self.prefix + self.correction_name, (self.outputs,), "vector"))
+        if self.bias_name:
+            specs.append(TensorSpec(self.prefix + self.bias_name, (self.outputs,), "vector"))
         for e in range(self.experts):
             g, u, d = self._names(e)
             specs += [TensorSpec(g, (F, H)), TensorSpec(u, (F, H)), TensorSpec(d, (H, F))]
@@ -87,6 +93,9 @@ class RoutedSwiGLU(FeedForward):
         self._bound = [self.router]
         if self.correction_name:
             self.correction = tensors[self.prefix + self.correction_name].to(torch.float32).contiguous()
+
+        if self.bias_name:
+            self.bias = tensors[self.prefix + self.bias_name].to(torch.float32).contiguous()
 
     def weight_bytes(self):
         # a step reads the router and, of the experts, what its tokens choose: at most every expert once
@@ -112,8 +121,8 @@ class RoutedSwiGLU(FeedForward):
         dest = torch.empty(P, dtype=torch.int32, device=dev)
         work = torch.empty(kernels.moe_work_size(P, E, tile), dtype=torch.int32, device=dev)
         xs = torch.empty((rows, self.hidden), dtype=x.dtype, device=dev) if tensor_cores else None
-        kernels.moe_route(ids, wts, perm, dest, work, x, self.router, batch.tok_seq, top, self.softmax_gate, self.renormalize, tile,
-                          xs=xs, apply_weight=self.weight_on_input, correction=self.correction, groups=self.groups,
+        kernels.moe_route(ids, wts, perm, dest, work, x, self.router, batch.tok_seq, top, gate=self.gate, renormalize=self.renormalize,
+                          tile_rows=tile, bias=self.bias, xs=xs, apply_weight=self.weight_on_input, correction=self.correction, groups=self.groups,
                           keep=self.keep, identity=self.identity, scale=self.scale, renorm_eps=self.renorm_eps,
                           group_best=self.group_best)
         a = torch.empty((rows, self.intermediate), dtype=x.dtype, device=dev)

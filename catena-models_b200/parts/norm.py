@@ -58,6 +58,52 @@ class ScalarRMSNorm(RMSNorm):
         self._bound = [self.weight]
 
 
+class LayerNorm(RMSNorm):
+    """y = (x - mean(x)) / sqrt(variance + eps) * w without a shift; the variance is the mean of the squared distances from
+    the mean.  Takes float32 rows (a float32 residual stream) and writes activations."""
+    fused_kind = "layer"
+
+    def apply(self, rt, x):
+        if x.dtype != torch.float32:
+            raise NotImplementedError("the layer norm reads float32 rows (ModelDefinition.residual_float32)")
+        y = torch.empty(x.shape, dtype=rt.dtype, device=x.device)
+        kernels.norm_f32in(y, x.contiguous(), self.weight, self.eps, layer=True)
+        return y
+
+
+class StreamNorm(LayerNorm):
+    """The layer norm of a weighted sum of hyper-connected streams: y = layer_norm(sum_s a_s X_s) for X [rows, S, width];
+    `read_name` names the tensor of the S factors, None: all are one (the end of the stack).  `open` makes the streams."""
+    fused_kind = "streams"
+
+    def __init__(self, name, width, eps, streams, read_name=None):
+        super().__init__(name, width, eps)
+        self.streams, self.read_name, self.read = int(streams), read_name, None
+
+    def tensor_specs(self):
+        return super().tensor_specs() + ([TensorSpec(self.read_name, (self.streams,), "vector")] if self.read_name else [])
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        if self.read_name:
+            self.read = tensors[self.read_name].to(torch.float32).contiguous()
+        else:
+            self.read = torch.ones(self.streams, dtype=torch.float32, device=self.weight.device)
+        self._bound.append(self.read)
+
+    def apply(self, rt, x):
+        n = torch.empty((x.shape[0], self.width), dtype=rt.dtype, device=x.device)
+        kernels.hyper_connect(x, n_out=n, read=self.read, w=self.weight, eps=self.eps)
+        return n
+
+    def open(self, rt, rows):
+        """(streams, this norm of them): every stream becomes `rows` [rows, width]."""
+        x = torch.empty((rows.shape[0], self.streams, self.width), dtype=torch.float32, device=rows.device)
+        n = torch.empty(rows.shape, dtype=rt.dtype, device=rows.device)
+        kernels.hyper_connect(rows, n_out=n, read=self.read, w=self.weight, eps=self.eps, out=x)
+        return x, n
+
+
 class DynamicTanh(Norm):
     """y = tanh(alpha x) * w + b in place of a norm: no mean, no variance, nothing that looks along the row.
     `alpha` is a learned scalar stored as `<name>.alpha`, the shift as `<name>.b`.  Takes float32 rows (a
@@ -91,4 +137,6 @@ class DynamicTanh(Norm):
 
 register_part("norm", "rms", RMSNorm)
 register_part("norm", "scalar_rms", ScalarRMSNorm)
+register_part("norm", "layer", LayerNorm)
+register_part("norm", "streams", StreamNorm)
 register_part("norm", "dynamic_tanh", DynamicTanh)

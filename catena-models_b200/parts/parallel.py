@@ -14,6 +14,9 @@ feed-forward, each sum with a constant factor.
 sublayers read the stream itself.  Optionally followed by an average over the depth of the stack: what the next layer
 reads is a weighted sum of the embedding output and of every layer's result so far.
 
+`HyperBlock`: the sequential arrangement on hyper-connected streams: the residual is several copies per token, a sublayer
+reads their weighted sum and its result is written back to all of them with a mix between them.
+
 `LoopEntry`: the step between two passes of a looped stack: h <- W [h; h0] + step, h0 being the embedding
 rows of the batch (the definition keeps them: `keep_embedding`) and `step` a learned row of the pass.  It
 has no norm of its own and no state; the product's float32 result becomes the new residual stream, and the
@@ -84,12 +87,12 @@ class ParallelBlock(Block):
 
 
 def _sum_and_norm(rt, h, terms, bias, next_norm):
-    """h += terms (+ bias); the next norm in the same kernel when it is an RMS norm or a dynamic tanh."""
+    """h += terms (+ bias); the next norm in the same kernel when it is an RMS norm, a layer norm or a dynamic tanh."""
     kind = getattr(next_norm, "fused_kind", None) if next_norm is not None else None
-    fuse = kind in ("rms", "dyt")
+    fuse = kind in ("rms", "dyt", "layer")
     n_out = torch.empty(h.shape, dtype=rt.dtype, device=h.device) if fuse else None
     kernels.residual_add_norm(h, terms, n_out, next_norm.weight if fuse else None, next_norm.eps if fuse else 0.0, bias,
-                              dyt=(next_norm.alpha, next_norm.shift) if kind == "dyt" else None)
+                              dyt=(next_norm.alpha, next_norm.shift) if kind == "dyt" else None, layer=kind == "layer")
     return h, n_out
 
 
@@ -206,6 +209,61 @@ class PostNormBlock(Block):
         return h, self._sum(rt, batch, h, f, self.ffn_norm, True, cast_last)
 
 
+class HyperBlock(Block):
+    """Two sublayers one after the other on hyper-connected streams X [rows, S, width] (float32).  Each sublayer f with its
+    norm reads u = sum_s a_s X_s and is written back as X_t <- sum_s M[s, t] X_s + c_t f(norm(u)).  `input_norm` and
+    `ffn_norm` are `streams` norms, which hold the factors a; `mixer_tensors` and `ffn_tensors` name M ([S, S], from, to) and c
+    ([S]) of either sublayer.  The feed-forward, its norm and its tensors may be absent together.  A write and the read of
+    whatever comes next are one kernel (`hyper_connect`)."""
+    prompt_capturable = True
+    supports_append = True
+
+    def __init__(self, mixer, feed_forward, input_norm, ffn_norm, streams, mixer_tensors, ffn_tensors=None):
+        if (feed_forward is None) != (ffn_norm is None) or (feed_forward is None) != (ffn_tensors is None):
+            raise ValueError("a feed-forward, its norm and its stream tensors come together")
+        if not 1 <= streams <= kernels.HYPER_MAX_STREAMS:
+            raise ValueError(f"HyperBlock: {streams} streams (1 to {kernels.HYPER_MAX_STREAMS})")
+        self.mixer, self.feed_forward, self.input_norm, self.ffn_norm = mixer, feed_forward, input_norm, ffn_norm
+        self.streams, self.names = streams, [n for n in (mixer_tensors, ffn_tensors) if n is not None]
+        self.writes = None
+
+    def children(self):
+        return [p for p in (self.input_norm, self.mixer, self.ffn_norm, self.feed_forward) if p is not None]
+
+    def tensor_specs(self):
+        S = self.streams
+        return [spec for mix, put in self.names for spec in (TensorSpec(mix, (S, S), "vector"), TensorSpec(put, (S,), "vector"))]
+
+    def bind(self, tensors, rt):
+        f32 = lambda name: tensors[name].to(torch.float32).contiguous()
+        self.writes = [(f32(mix), f32(put)) for mix, put in self.names]
+        self._bound = [t for pair in self.writes for t in pair]
+
+    def state_spec(self):
+        return self.mixer.state_spec()
+
+    def _write(self, rt, x, y, which, reader):
+        """The sublayer's result into the streams; the reader's normed rows when it reads streams."""
+        mix, put = self.writes[which]
+        fuse = getattr(reader, "fused_kind", None) == "streams"
+        n = torch.empty((x.shape[0], x.shape[2]), dtype=rt.dtype, device=x.device) if fuse else None
+        kernels.hyper_connect(x, _terms(y), mix, put, n_out=n, read=reader.read if fuse else None,
+                              w=reader.weight if fuse else None, eps=reader.eps if fuse else 0.0)
+        return x, n
+
+    def forward(self, rt, batch, h, n, state, next_norm):
+        if h.dim() != 3 or h.dtype != torch.float32:
+            raise ValueError("HyperBlock works on float32 streams (ModelDefinition.streams)")
+        batch.partial_sums_ok = False
+        if n is None:
+            n = self.input_norm.apply(rt, h)
+        y = self.mixer.forward(rt, batch, n, state)
+        if self.feed_forward is None:
+            return self._write(rt, h, y, 0, next_norm)
+        h, n2 = self._write(rt, h, y, 0, self.ffn_norm)
+        return self._write(rt, h, self.feed_forward.forward(rt, batch, n2), 1, next_norm)
+
+
 class LoopEntry(Block):
     prompt_capturable = True
     supports_append = True
@@ -236,4 +294,5 @@ register_part("mixer", "side_by_side", SideBySide)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "postnorm", PostNormBlock)
+register_part("block", "hyper", HyperBlock)
 register_part("block", "loop_entry", LoopEntry)

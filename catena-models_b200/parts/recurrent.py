@@ -20,8 +20,8 @@ a running maximum m that starts at 0
 
 then the same unit norm, channel weight, sigmoid(W_g h) gate and output projection.  State: S, n, m, float32.
 
-`GatedDecayMemory` (gated linear attention) and `ConstantDecayMemory` (lightning attention) are described at their
-classes.
+`GatedDecayMemory` (gated linear attention), `ConstantDecayMemory` (lightning attention) and `DeltaRule` (gated delta
+rule) are described at their classes.
 
 Decays, gates, exponentials, the state and every sum over it are float32 whatever the activation dtype;
 the projections run through the runtime's products.  Both mixers run every kind of step through one
@@ -260,7 +260,68 @@ class GatedDecayMemory(Mixer):
         return self.out.apply(rt, o, out_dtype=self.out_dtype)
 
 
+class DeltaRule(Mixer):
+    """Gated delta rule: q, k (kv_heads x dim) and v (heads x value_dim) pass a short causal filter per channel (`taps` taps,
+    stored as `<name>.conv` [channels, taps], the last one the present token's) and silu; q and k become unit vectors
+    x / sqrt(sum x^2 + unit_eps), q times 1 / sqrt(dim); head h uses q/k head h / (heads / kv_heads).  With
+    beta = sigmoid(W_b h) and g = exp(-exp(A_log) softplus(W_a h + dt_bias)), both one number per head:
+
+        S <- g S        u = beta (v - S^T k)        S <- S + k u^T        o = S^T q
+
+    Each head's o is brought to unit root mean square over its value channels, times a weight per value channel that all
+    heads share, times silu(W_g h), then the output projection.  State per sequence: S and the filter's last inputs, float32.
+
+    Single tokens run filter, gates, recurrence, norm and output gate of a head as one kernel (where the head sizes allow);
+    longer steps form all rows' inputs side by side, then walk the recurrence (csrc/delta.cu)."""
+    prompt_capturable = True
+    supports_append = True
+
+    def __init__(self, prefix, hidden, heads, kv_heads, dim, value_dim, taps, eps, unit_eps=1e-6, out_dtype=None):
+        if heads % kv_heads or taps < 1:
+            raise ValueError(f"DeltaRule: {heads} heads over {kv_heads}, {taps} taps")
+        self.prefix, self.hidden, self.heads, self.kv_heads = prefix, hidden, heads, kv_heads
+        self.dim, self.value_dim, self.taps, self.eps, self.unit_eps = dim, value_dim, taps, float(eps), float(unit_eps)
+        self.k_size, self.v_size = kv_heads * dim, heads * value_dim
+        self.qkvg = Linear([prefix + s for s in "qkvg"], [self.k_size, self.k_size, self.v_size, self.v_size], hidden)
+        self.gates = Linear([prefix + "b", prefix + "a"], [heads, heads], hidden)
+        self.out = Linear(prefix + "o", hidden, self.v_size)
+        self.out_dtype = {None: None, "float32": torch.float32}[out_dtype]
+
+    def children(self):
+        return [self.qkvg, self.gates, self.out]
+
+    def tensor_specs(self):
+        p, K = self.prefix, self.taps
+        return [TensorSpec(p + "q.conv", (self.k_size, K), "conv"), TensorSpec(p + "k.conv", (self.k_size, K), "conv"),
+                TensorSpec(p + "v.conv", (self.v_size, K), "conv"), TensorSpec(p + "A_log", (self.heads,), "vector"),
+                TensorSpec(p + "dt_bias", (self.heads,), "vector"), TensorSpec(p + "norm", (self.value_dim,), "norm")]
+
+    def bind(self, tensors, rt):
+        p = self.prefix
+        f32 = lambda name: tensors[p + name].to(torch.float32).contiguous()
+        self.tap_w = torch.cat([f32("q.conv"), f32("k.conv"), f32("v.conv")]).contiguous()
+        self.rate, self.dt_bias = torch.exp(f32("A_log")), f32("dt_bias")
+        self.norm_w = f32("norm").repeat(self.heads).contiguous()              # the norm kernel indexes head x channel
+        self._bound = [self.tap_w, self.rate, self.dt_bias, self.norm_w]
+        self.one_kernel = kernels.delta_step_fits(self.dim, self.value_dim)
+
+    def state_spec(self):
+        return FixedStateSpec((kernels.delta_state_floats(self.heads, self.kv_heads, self.dim, self.value_dim, self.taps),), "float32")
+
+    def forward(self, rt, batch, x, state):
+        proj = self.qkvg.apply(rt, x)
+        o = torch.empty((batch.T, self.v_size), dtype=x.dtype, device=x.device)
+        if batch.kind == "decode" and self.one_kernel:
+            inputs = {"x": x, "w_gates": self.gates.weight}
+        else:
+            inputs = {"gates": self.gates.apply(rt, x, out_dtype=torch.float32)}
+        kernels.delta_rule(o, proj, self.tap_w, self.rate, self.dt_bias, self.norm_w, state.tensor, batch, self.heads, self.kv_heads,
+                           self.dim, self.value_dim, self.dim ** -0.5, self.unit_eps, self.eps, **inputs)
+        return self.out.apply(rt, o, out_dtype=self.out_dtype)
+
+
 register_part("mixer", "decay_mix", DecayMix)
+register_part("mixer", "delta_rule", DeltaRule)
 register_part("mixer", "gated_decay_memory", GatedDecayMemory)
 register_part("mixer", "constant_decay_memory", ConstantDecayMemory)
 register_part("mixer", "matrix_memory", MatrixMemory)
