@@ -602,6 +602,21 @@ def relilix_config(size, vocab=VOCAB):
                 layers=layers)
 
 
+def kofadra_config(size, vocab=VOCAB):
+    """For `--compare kofadra`: six layers of the Kofadra decoder, the middle two run twice, at the same width, heads and
+    expert width as the Narasun model above: in turn a gated delta rule (the matrix memory's heads and head sizes, half as
+    many q/k heads, four taps) and an attention (the attention's heads, chunks of 1,024 positions), each with a routed
+    feed-forward, on four hyper-connected streams."""
+    z = COMPARE_SIZES[size]
+    moe = dict(kind="moe", expert=dict(ff=z["expert_ff"]), router=dict(experts=z["experts"], top=z["top"]))
+    delta = dict(type="delta", mlp=moe, mixer=dict(heads=z["mem_heads"], kv_heads=z["mem_heads"] // 2, dim=z["mem_dim"],
+                                                   vdim=z["mem_vdim"], conv=4))
+    att = dict(type="attention", mlp=moe, mixer=dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["head"], vdim=z["head"],
+                                                     scale=z["head"] ** -0.5, mask=dict(size=1024)))
+    return dict(architecture="Kofadra", vocab=vocab, width=z["width"], norm=dict(eps=1e-6), embedding=dict(scale=z["width"] ** 0.5),
+                streams=4, layers=[delta, att] * 3, loop=dict(start=2, stop=4, times=2))
+
+
 def latent_decode_table(pk, device="cuda:0", cases=((8, 16, 256, 32), (128, 16, 256, 32), (64, 32, 512, 32)), held=2048):
     """`--latent-table`: the single-token latent attention alone, in its tensor-core and its CUDA-core form: `B` sequences
     that hold `held` tokens, `H` heads over latents of `KR` + `R` channels, random bfloat16 entries in pages laid out in
@@ -717,7 +732,7 @@ def _kernel_rows(torch, model, prompt_len, batch, vocab):
 def compare_designs(which, sizes, prompt_len, batch, steps, pk, tables):
     """Prefill and decode throughput of a design beside the closest earlier one at equal size, random weights: the
     Narasun decoder beside an LFM3 decoder, the Fozedra and the Maferax decoder beside the Narasun decoder, the Relilix
-    decoder beside the Maferax decoder."""
+    decoder beside the Maferax decoder, the Kofadra decoder beside the Narasun and the Maferax decoder."""
     import torch
 
     from catena_models_b200.api import Model
@@ -732,7 +747,8 @@ def compare_designs(which, sizes, prompt_len, batch, steps, pk, tables):
         pairs = {"narasun": (("Narasun", narasun_config), ("LFM3", lfm3_like_config)),
                  "fozedra": (("Fozedra", fozedra_config), ("Narasun", narasun_config)),
                  "maferax": (("Maferax", maferax_config), ("Narasun", narasun_config)),
-                 "relilix": (("Relilix", relilix_config), ("Maferax", maferax_config))}[which]
+                 "relilix": (("Relilix", relilix_config), ("Maferax", maferax_config)),
+                 "kofadra": (("Kofadra", kofadra_config), ("Narasun", narasun_config), ("Maferax", maferax_config))}[which]
         for name, cfg in ((n, make(size, vocab)) for n, make in pairs):
             model = Model.random(cfg, seed=0, std=0.02, dtype="bfloat16", max_tokens=batch * (prompt_len + 256) + 4096,
                                  max_seqs=batch + 1)
@@ -774,7 +790,7 @@ def main():
                     help="time the prompt-attention kernels alone at 2,048, 4,096 and 16,384 tokens and print the table")
     ap.add_argument("--latent-table", action="store_true",
                     help="instead of the JSON line: time the single-token latent attention alone, tensor-core and CUDA-core form")
-    ap.add_argument("--compare", default=None, choices=["narasun", "fozedra", "maferax", "relilix"],
+    ap.add_argument("--compare", default=None, choices=["narasun", "fozedra", "maferax", "relilix", "kofadra"],
                     help="instead of the JSON line: prompt and decode throughput of that design beside the closest earlier "
                          "one at equal size (random weights: Narasun beside LFM3, Fozedra and Maferax beside Narasun, Relilix beside "
                          "Maferax), as a table")

@@ -14,7 +14,8 @@
 //
 // Steps of one token per sequence run delta_step_kernel: everything from the filter to the gated output of a head in one
 // block.  Longer steps run delta_prepare_kernel (filter, silu, unit vectors, gates: all rows side by side), then the
-// recurrence row by row (delta_scan_kernel), then norm and gate (cm_scan_norm_gate).
+// recurrence: row by row (delta_scan_kernel) with norm and gate behind it (cm_scan_norm_gate), or, for long steps, in
+// chunks of rows (delta_chunk.cu).
 #include "common.cuh"
 #include "delta.h"
 #include "recurrent.h"
@@ -324,6 +325,7 @@ static int delta_prompt(const DeltaArgs& a, cudaStream_t st) {
         cm_launch(delta_ring_kernel<T>, dim3((C + 127) / 128, a.B), 128, 0, st, a);
         CM_CHECK_LAUNCH();
     }
+    if (a.chunks) return delta_chunked<T>(a, st);
     const int rc = launch_delta_scan<T>(a, st);
     if (rc != CM_OK) return rc;
     ScanArgs n = {};

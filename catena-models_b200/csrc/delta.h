@@ -29,3 +29,7 @@ struct DeltaArgs {
     float* chunks;                // scratch of the chunked form, or null: the serial scan
     int max_len;                  // most rows that a sequence brings
 };
+
+// The recurrence of a step with norm and gate, in chunks (delta_chunk.cu); a.chunks is its scratch.
+template <typename T>
+int delta_chunked(const DeltaArgs& a, cudaStream_t st);

@@ -1013,13 +1013,24 @@ def delta_state_floats(H, G, D, DV, K):
     return -(-(H * D * DV + (K * (2 * G * D + H * DV) if K > 1 else 0)) // 4) * 4
 
 
+def delta_chunk_floats(B, max_len, H, D, DV):
+    """Floats of scratch that the chunked form of `delta_rule` takes for B sequences of up to max_len rows; 0: it does not
+    take heads of D x DV."""
+    fn = lib().cm_delta_chunk_floats
+    fn.argtypes, fn.restype = [_i, _i, _i, _i, _i], _ll
+    return fn(B, max_len, H, D, DV)
+
+
 def delta_rule(out, proj, taps, rate, dt_bias, norm_w, state, batch, H, G, D, DV, q_scale, unit_eps, eps, gates=None, x=None,
-               w_gates=None):
+               w_gates=None, chunk_scratch=None):
     """The gated delta rule behind its projections (csrc/delta.cu).  proj [rows, n]: q (G D channels) | k (G D) | v (H DV) |
     output gate (H DV), activation dtype; taps float32 [2 G D + H DV, K]; rate, dt_bias float32 [H]; norm_w float32 [H DV];
     state float32 [slots, delta_state_floats]; out [rows, H DV].  `gates` float32 [rows, >= 2 H]: the pre-activations of
     beta, then of the decay, for a step of any lengths; or, for a step of one token per sequence whose heads fit
-    (`delta_step_fits`), the mixer's input `x` [rows, W] and the gate projections' rows `w_gates` [2 H, W]: one kernel."""
+    (`delta_step_fits`), the mixer's input `x` [rows, W] and the gate projections' rows `w_gates` [2 H, W]: one kernel.
+    `chunk_scratch` (float32, at least `delta_chunk_floats` elements): the recurrence in chunks of 64 rows, of which only the
+    state's step from chunk to chunk is serial (csrc/delta_chunk.cu); its numbers agree with the row-by-row form's beyond
+    rounding."""
     rows, C, K = proj.shape[0], 2 * G * D + H * DV, taps.shape[1]
     if taps.shape[0] != C or proj.shape[1] < C + H * DV or proj.stride(1) != 1 or out.dtype != proj.dtype or out.stride(1) != 1:
         raise KernelError("delta_rule: the projected rows do not hold the channels that the taps name")
@@ -1049,8 +1060,13 @@ def delta_rule(out, proj, taps, rate, dt_bias, norm_w, state, batch, H, G, D, DV
     lb = torch.empty((rows, 2 * H), dtype=torch.float32, device=proj.device)
     raw = torch.empty((rows, H * DV), dtype=torch.float32, device=proj.device)
     a.gates, a.ldg, a.qk, a.v, a.lb, a.raw = _ptr(gates), gates.stride(0), _ptr(qk), _ptr(v), _ptr(lb), _ptr(raw)
-    _check(lib().cm_delta_prompt(dtype_code(proj.dtype), ctypes.byref(a), _stream()), "delta_prompt",
-           3 if K < 2 or a.from_zero else 4,
+    if chunk_scratch is not None:
+        need = delta_chunk_floats(batch.B, batch.max_len, H, D, DV)
+        if need < 1 or chunk_scratch.dtype != torch.float32 or chunk_scratch.numel() < need or chunk_scratch.data_ptr() % 16:
+            raise KernelError("delta_rule: the chunked form does not take these heads, or its scratch is short")
+        a.chunks = _ptr(chunk_scratch)
+    _check(lib().cm_delta_prompt(dtype_code(proj.dtype), ctypes.byref(a), _stream()), "delta_chunked" if chunk_scratch is not None else "delta_prompt",
+           (3 if K < 2 or a.from_zero else 4) + int(chunk_scratch is not None),
            cost=lambda: (f"{batch.B} sequences, {rows} rows, {H}/{G} heads of {D}x{DV}, {K} taps", moved, flops))
 
 

@@ -272,9 +272,12 @@ class DeltaRule(Mixer):
     heads share, times silu(W_g h), then the output projection.  State per sequence: S and the filter's last inputs, float32.
 
     Single tokens run filter, gates, recurrence, norm and output gate of a head as one kernel (where the head sizes allow);
-    longer steps form all rows' inputs side by side, then walk the recurrence (csrc/delta.cu)."""
+    longer steps form all rows' inputs side by side, then walk the recurrence row by row (csrc/delta.cu) or, from
+    CHUNKED_MIN_ROWS rows a sequence on, in chunks of 64 rows (csrc/delta_chunk.cu)."""
     prompt_capturable = True
     supports_append = True
+    CHUNKED_MIN_ROWS = 48                   # shorter steps walk row by row
+    CHUNKED_MAX_SCRATCH = 512 << 20         # bytes of per-chunk matrices above which a step walks row by row
 
     def __init__(self, prefix, hidden, heads, kv_heads, dim, value_dim, taps, eps, unit_eps=1e-6, out_dtype=None):
         if heads % kv_heads or taps < 1:
@@ -315,6 +318,10 @@ class DeltaRule(Mixer):
             inputs = {"x": x, "w_gates": self.gates.weight}
         else:
             inputs = {"gates": self.gates.apply(rt, x, out_dtype=torch.float32)}
+            if batch.kind != "decode" and batch.max_len >= self.CHUNKED_MIN_ROWS:
+                need = kernels.delta_chunk_floats(batch.B, batch.max_len, self.heads, self.dim, self.value_dim)
+                if 0 < need * 4 <= self.CHUNKED_MAX_SCRATCH:
+                    inputs["chunk_scratch"] = rt.scratch("delta_chunks", need)
         kernels.delta_rule(o, proj, self.tap_w, self.rate, self.dt_bias, self.norm_w, state.tensor, batch, self.heads, self.kv_heads,
                            self.dim, self.value_dim, self.dim ** -0.5, self.unit_eps, self.eps, **inputs)
         return self.out.apply(rt, o, out_dtype=self.out_dtype)
