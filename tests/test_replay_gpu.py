@@ -217,6 +217,25 @@ def test_replay_of_a_relilix_model(tmp_path, name, dtype):
     _replay_whole_tail_and_together(tmp_path, folder, V, reqs, exact, exact, dtype)
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "M"])
+def test_replay_of_a_kofadra_model(tmp_path, name, dtype):
+    """The sixth architecture through the same program, on the same schedule (chunks that end in prompts and in decoding,
+    states of every pass of a loop); bfloat16 as for the fifth."""
+    import plain_kofadra
+    import tiny_kofadra
+
+    folder = tiny_kofadra.make_folder(tmp_path, name, seed=7)
+    cfg, tensors = tiny_kofadra.load_plain(folder)
+    V = cfg["vocab"]
+    reqs = {k: tiny_kofadra.prompt(n, V, seed=ord(k)) for k, n in {"a": 1, "b": 70, "c": 135, "d": 90}.items()}
+    if dtype == "bfloat16":
+        _replay_whole_tail_and_together(tmp_path, folder, V, reqs, None, None, dtype, against_library=True)
+        return
+    exact = {k: plain_kofadra.forward(t, tensors, cfg)[0] for k, t in reqs.items()}
+    _replay_whole_tail_and_together(tmp_path, folder, V, reqs, exact, exact, dtype)
+
+
 def _library_steps(folder, dtype, steps, max_tokens):
     """The same schedule through the library's engine in this process: {step: logits of its wanted places}."""
     from catena_models_b200.api import Model
