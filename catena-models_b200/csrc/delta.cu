@@ -53,7 +53,10 @@ __device__ __forceinline__ float2 two_of(const float* p, bool pair, bool second)
 
 // A warp takes one unit of a row: a head of q, a head of k, or a run of up to 64 NP channels of v; lane l owns the channels
 // 2 l, 2 l + 1 of every 64.  Units [0, G): q heads; [G, 2 G): k heads; then the runs of v; the last unit is the gates.
-template <typename T, int NP>
+// Where the warp's rows all belong to one sequence, and every tap of all of them lies in the step (the usual case of a long
+// prompt), the rows' inputs are fetched once, side by side, and the taps of a channel stay in registers (KF > 0: K = KF taps;
+// 0: the general form alone).
+template <typename T, int NP, int KF>
 __global__ void __launch_bounds__(32 * DP_WARPS)
 delta_prepare_kernel(const DeltaArgs a, int v_units, int pairs_ok) {
     pdl_trigger();
@@ -75,6 +78,74 @@ delta_prepare_kernel(const DeltaArgs a, int v_units, int pairs_ok) {
     const bool is_v = unit >= 2 * G;
     const int c0 = is_v ? 2 * G * D + (unit - 2 * G) * 64 * NP : unit * D;       // first channel of the unit
     const int n = is_v ? min(64 * NP, C - c0) : D;
+    if constexpr (KF > 0) {
+        const long long t_last = t_first + DP_TOKENS - 1;
+        int b = -1;
+        bool fast = pairs_ok && t_last < a.rows;
+        if (fast) {
+            b = a.tok_seq[t_first];
+            fast = b >= 0 && a.tok_seq[t_last] == b && a.tok_pos[t_first] - (KF - 1) >= a.seq_pos0[b];
+        }
+        if (fast) {
+            const int last = a.seq_pos0[b] + a.seq_start[b + 1] - a.seq_start[b] - (KF - 1), pos = a.tok_pos[t_first];
+            float* ring = KF > 1 ? delta_ring(a, a.seq_slot[b]) : nullptr;
+            float y[DP_TOKENS][NP][2], ss[DP_TOKENS];
+#pragma unroll
+            for (int i = 0; i < DP_TOKENS; ++i) ss[i] = 0.f;
+#pragma unroll
+            for (int p = 0; p < NP; ++p) {
+                const int c = 64 * p + 2 * lane;
+                if (c >= n) continue;                          // n is even here
+                float2 u[DP_TOKENS + KF - 1];
+                const T* src = (const T*)a.proj + (t_first - (KF - 1)) * a.ldp + c0 + c;
+#pragma unroll
+                for (int r = 0; r < DP_TOKENS + KF - 1; ++r) u[r] = two_of(src + (long long)r * a.ldp, true, true);
+                float w0[KF], w1[KF];
+#pragma unroll
+                for (int j = 0; j < KF; ++j) {
+                    w0[j] = a.taps[(long long)(c0 + c) * KF + j];
+                    w1[j] = a.taps[(long long)(c0 + c + 1) * KF + j];
+                }
+#pragma unroll
+                for (int i = 0; i < DP_TOKENS; ++i) {
+                    float y0 = 0.f, y1 = 0.f;
+#pragma unroll
+                    for (int j = 0; j < KF; ++j) {
+                        y0 = fmaf(w0[j], u[i + j].x, y0);
+                        y1 = fmaf(w1[j], u[i + j].y, y1);
+                    }
+                    if (KF > 1 && a.from_zero && pos + i >= last)
+                        *reinterpret_cast<float2*>(ring + (long long)((pos + i) % KF) * C + c0 + c) = u[i + KF - 1];
+                    y[i][p][0] = silu_f32(y0);
+                    y[i][p][1] = silu_f32(y1);
+                    ss[i] = fmaf(y[i][p][0], y[i][p][0], fmaf(y[i][p][1], y[i][p][1], ss[i]));
+                }
+            }
+            if (!is_v) {
+#pragma unroll
+                for (int i = 0; i < DP_TOKENS; ++i) ss[i] = (unit < G ? a.q_scale : 1.f) / sqrtf(warp_sum(ss[i]) + a.unit_eps);
+            }
+#pragma unroll
+            for (int p = 0; p < NP; ++p) {
+                const int c = 64 * p + 2 * lane;
+                if (c >= n) continue;
+#pragma unroll
+                for (int i = 0; i < DP_TOKENS; ++i) {
+                    const long long t = t_first + i;
+                    if (is_v) {
+                        T* dst = (T*)a.v + t * (long long)a.H * a.DV + (c0 - 2 * G * D) + c;
+                        if constexpr (sizeof(T) == 2)
+                            *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(y[i][p][0], y[i][p][1]);
+                        else
+                            *reinterpret_cast<float2*>(dst) = make_float2(y[i][p][0], y[i][p][1]);
+                    } else {
+                        *reinterpret_cast<float2*>(a.qk + t * 2 * G * D + c0 + c) = make_float2(y[i][p][0] * ss[i], y[i][p][1] * ss[i]);
+                    }
+                }
+            }
+            return;
+        }
+    }
     for (int i = 0; i < DP_TOKENS; ++i) {
         const long long t = t_first + i;
         if (t >= a.rows) return;
@@ -308,18 +379,30 @@ static int delta_check(const DeltaArgs& a) {
 template <typename T>
 static int delta_prompt(const DeltaArgs& a, cudaStream_t st) {
     const int C = delta_channels(a), vw = a.H * a.DV;
-    const bool pairs = a.D % 2 == 0 && a.ldp % 2 == 0 && ((uintptr_t)a.proj & (2 * sizeof(T) - 1)) == 0;
-#define DP_LAUNCH(NP)                                                                                                    \
+    const bool pairs = a.D % 2 == 0 && vw % 2 == 0 && a.ldp % 2 == 0 && a.state_stride % 2 == 0 && (a.H * a.D * a.DV) % 2 == 0 &&
+                       (((uintptr_t)a.proj | (uintptr_t)a.v) & (2 * sizeof(T) - 1)) == 0 &&
+                       (((uintptr_t)a.qk | (uintptr_t)a.state) & 7) == 0;
+#define DP_LAUNCH(NP) DP_LAUNCH_K(NP, 0)
+#define DP_LAUNCH_K(NP, KF)                                                                                                    \
     do {                                                                                                                 \
         const int v_units = (vw + 64 * NP - 1) / (64 * NP);                                                              \
         dim3 grid((unsigned)((a.rows + DP_WARPS * DP_TOKENS - 1) / (DP_WARPS * DP_TOKENS)), 2 * a.G + v_units + 1);       \
-        cm_launch(delta_prepare_kernel<T, NP>, grid, 32 * DP_WARPS, 0, st, a, v_units, (int)(pairs && vw % 2 == 0));      \
+        cm_launch(delta_prepare_kernel<T, NP, KF>, grid, 32 * DP_WARPS, 0, st, a, v_units, (int)pairs);                   \
     } while (0)
-    if (a.D <= 64) DP_LAUNCH(1);
-    else if (a.D <= 128) DP_LAUNCH(2);
+#define DP_CASES(NP)                            \
+    do {                                        \
+        if (a.K == 2) DP_LAUNCH_K(NP, 2);       \
+        else if (a.K == 3) DP_LAUNCH_K(NP, 3);  \
+        else if (a.K == 4) DP_LAUNCH_K(NP, 4);  \
+        else DP_LAUNCH(NP);                     \
+    } while (0)
+    if (a.D <= 64) DP_CASES(1);
+    else if (a.D <= 128) DP_CASES(2);
     else if (a.D <= 256) DP_LAUNCH(4);
     else DP_LAUNCH(16);
+#undef DP_CASES
 #undef DP_LAUNCH
+#undef DP_LAUNCH_K
     CM_CHECK_LAUNCH();
     if (a.K > 1 && !a.from_zero) {
         cm_launch(delta_ring_kernel<T>, dim3((C + 127) / 128, a.B), 128, 0, st, a);
@@ -364,7 +447,7 @@ template <typename T, int NR>
 __global__ void __launch_bounds__(512)
 delta_step_kernel(const DeltaArgs a, int RS) {
     extern __shared__ __align__(16) float sm[];
-    __shared__ float red[5][32];
+    __shared__ float red[2][32];
     pdl_trigger();
     pdl_wait();
     const int hd = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, NT = blockDim.x, lane = tid & 31, warp = tid >> 5;
@@ -391,8 +474,8 @@ delta_step_kernel(const DeltaArgs a, int RS) {
     float* ring = K > 1 ? delta_ring(a, slot) : nullptr;
     const T* src = (const T*)a.proj + t * a.ldp;
     const bool own_qk = hd % (H / G) == 0;
-    float sqq = 0.f, skk = 0.f, sqk = 0.f, zb = 0.f, za = 0.f;
-    auto filtered = [&](int c, bool keep) {
+    for (int e = tid; e < 2 * D + DV; e += NT) {
+        const int c = e < D ? kh * D + e : (e < 2 * D ? G * D + kh * D + e - D : 2 * G * D + hd * DV + e - 2 * D);
         const float* w = a.taps + (long long)c * K;
         const float now = to_f32(src[c]);
         float y = 0.f;
@@ -400,40 +483,59 @@ delta_step_kernel(const DeltaArgs a, int RS) {
             const int s = pos - K + 1 + j;
             y = fmaf(w[j], s >= 0 ? ring[(long long)(s % K) * C + c] : 0.f, y);
         }
-        if (keep && K > 1) ring[(long long)(pos % K) * C + c] = now;
-        return silu_f32(fmaf(w[K - 1], now, y));
-    };
-    for (int i = tid; i < D; i += NT) {
-        const float q = filtered(kh * D + i, own_qk), k = filtered(G * D + kh * D + i, own_qk);
-        qs[i] = q;
-        ks[i] = k;
-        sqq = fmaf(q, q, sqq);
-        skk = fmaf(k, k, skk);
-        sqk = fmaf(q, k, sqk);
+        y = silu_f32(fmaf(w[K - 1], now, y));
+        if (K > 1 && (own_qk || e >= 2 * D)) ring[(long long)(pos % K) * C + c] = now;
+        if (e < D) qs[e] = y;
+        else if (e < 2 * D) ks[e - D] = y;
+        else vs[e - 2 * D] = rounded<T>(y);
     }
-    for (int j = tid; j < DV; j += NT) vs[j] = rounded<T>(filtered(2 * G * D + hd * DV + j, true));
+    float zb = 0.f, za = 0.f;                          // the gates' projections
     {
         const T* xr = (const T*)a.x + t * a.W;
         const T* wb = (const T*)a.w_gates + (long long)hd * a.W;
         const T* wa = (const T*)a.w_gates + (long long)(H + hd) * a.W;
-        for (int c = tid; c < a.W; c += NT) {
-            const float x = to_f32(xr[c]);
-            zb = fmaf(to_f32(wb[c]), x, zb);
-            za = fmaf(to_f32(wa[c]), x, za);
-        }
-    }
-    float sums[5] = {sqq, skk, sqk, zb, za};
+        if (a.W % 8 == 0 && ((((uintptr_t)a.x) | ((uintptr_t)a.w_gates)) & 15) == 0) {
+            for (int c = tid * 8; c < a.W; c += NT * 8) {
+                float x[8], u[8], v[8];
+                load8f<T>(xr + c, x);
+                load8f<T>(wb + c, u);
+                load8f<T>(wa + c, v);
 #pragma unroll
-    for (int i = 0; i < 5; ++i) {
-        sums[i] = warp_sum(sums[i]);
-        if (lane == 0) red[i][warp] = sums[i];
+                for (int i = 0; i < 8; ++i) {
+                    zb = fmaf(u[i], x[i], zb);
+                    za = fmaf(v[i], x[i], za);
+                }
+            }
+        } else {
+            for (int c = tid; c < a.W; c += NT) {
+                const float x = to_f32(xr[c]);
+                zb = fmaf(to_f32(wb[c]), x, zb);
+                za = fmaf(to_f32(wa[c]), x, za);
+            }
+        }
+        zb = warp_sum(zb);
+        za = warp_sum(za);
+        if (lane == 0) {
+            red[0][warp] = zb;
+            red[1][warp] = za;
+        }
     }
     __syncthreads();
     const int nw = NT >> 5;
-#pragma unroll
-    for (int i = 0; i < 5; ++i) sums[i] = warp_sum(lane < nw ? red[i][lane] : 0.f);
-    const float fq = a.q_scale / sqrtf(sums[0] + a.unit_eps), fk = 1.f / sqrtf(sums[1] + a.unit_eps);
-    const float g = expf(log_decay_of(a, hd, sums[4])), beta = sigmoid_f32(sums[3]), qk = sums[2] * fq * fk;
+    zb = warp_sum(lane < nw ? red[0][lane] : 0.f);
+    za = warp_sum(lane < nw ? red[1][lane] : 0.f);
+    float sqq = 0.f, skk = 0.f, sqk = 0.f;             // every warp forms them for itself
+    for (int i = lane; i < D; i += 32) {
+        const float q = qs[i], k = ks[i];
+        sqq = fmaf(q, q, sqq);
+        skk = fmaf(k, k, skk);
+        sqk = fmaf(q, k, sqk);
+    }
+    sqq = warp_sum(sqq);
+    skk = warp_sum(skk);
+    sqk = warp_sum(sqk);
+    const float fq = a.q_scale / sqrtf(sqq + a.unit_eps), fk = 1.f / sqrtf(skk + a.unit_eps);
+    const float g = expf(log_decay_of(a, hd, za)), beta = sigmoid_f32(zb), qk = sqk * fq * fk;
     if (mine) {
         float4 dk = make_float4(0.f, 0.f, 0.f, 0.f), dq = dk;
 #pragma unroll

@@ -28,6 +28,7 @@ struct DeltaChunkGeom {
     int D4, DV4;                 // D and DV rounded up to multiples of 4
     int chunks;                  // chunks per sequence that the launch provides for
     int NCp;                     // pitch of [W | U]
+    int stages;                  // chunks whose M^T and N pass 2 holds at a time
     long long stride;            // floats of one chunk of one head in the scratch: M^T [D4][D4], N [D4][DV4], Q'^T [D4][DC]
 };
 
@@ -37,6 +38,7 @@ static __host__ __device__ __forceinline__ DeltaChunkGeom delta_chunk_geom(int D
     g.DV4 = (DV + 3) & ~3;
     g.chunks = (max_len + DC - 1) / DC;
     g.NCp = g.D4 + g.DV4 + 4;
+    g.stages = g.D4 <= 64 ? 4 : (g.D4 <= 96 ? 3 : 2);
     g.stride = (long long)g.D4 * (g.D4 + g.DV4 + DC);
     return g;
 }
@@ -45,7 +47,7 @@ static size_t delta_chunk_smem(const DeltaChunkGeom& g) {
     return ((first > x ? first : x) + (size_t)DC * (g.D4 + 4) + 2 * DC * DC_LD + 4 * DC) * sizeof(float);
 }
 static size_t delta_walk_smem(const DeltaChunkGeom& g) {
-    return ((size_t)2 * g.D4 * g.D4 + 2 * g.D4 * DC_COLS + (size_t)g.D4 * DC_COLS + DC_THREADS * 16) * sizeof(float);
+    return ((size_t)g.stages * g.D4 * (g.D4 + 4 + DC_COLS) + 2 * (size_t)g.D4 * DC_COLS) * sizeof(float);
 }
 static size_t delta_read_smem(const DeltaChunkGeom& g) { return ((size_t)g.D4 * DC_LD + (size_t)g.D4 * DC_LD) * sizeof(float); }
 
@@ -64,6 +66,12 @@ __device__ __forceinline__ void tile_mac(float (&acc)[4][4], const float* A, int
 #pragma unroll
             for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xs[i], ys[j], acc[i][j]);
     }
+}
+// two sums at once: u += a w, v += b w (one instruction on register pairs)
+__device__ __forceinline__ void fma_two(float& u, float& v, float a, float b, float w) {
+    asm("{\n\t.reg .b64 p, q, r;\n\tmov.b64 p, {%0, %1};\n\tmov.b64 q, {%2, %3};\n\tmov.b64 r, {%4, %4};\n\t"
+        "fma.rn.f32x2 p, q, r, p;\n\tmov.b64 {%0, %1}, p;\n\t}"
+        : "+f"(u), "+f"(v) : "f"(a), "f"(b), "f"(w));
 }
 __device__ __forceinline__ void tile_zero(float (&acc)[4][4]) {
 #pragma unroll
@@ -197,10 +205,8 @@ delta_chunk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
 #pragma unroll
             for (int t = (s + 1) & ~3; t < DC; t += 4) {                // A_ts is zero for t <= s
                 const float4 A = *reinterpret_cast<const float4*>(AT + s * DC_LD + t);
-                x[t] = fmaf(A.x, xs, x[t]);
-                x[t + 1] = fmaf(A.y, xs, x[t + 1]);
-                x[t + 2] = fmaf(A.z, xs, x[t + 2]);
-                x[t + 3] = fmaf(A.w, xs, x[t + 3]);
+                fma_two(x[t], x[t + 1], A.x, A.y, xs);
+                fma_two(x[t + 2], x[t + 3], A.z, A.w, xs);
             }
         }
 #pragma unroll
@@ -271,9 +277,12 @@ __device__ __forceinline__ void dc_copy16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
-// A block owns DC_COLS columns of one head's S for one sequence.  S lies in shared memory; M^T and N of the next chunk are on
-// their way while the present one is multiplied.  The sum over a row of M is dealt to `parts` groups of threads (tiles of
-// 4 x 4), whose shares are added in order.  N's place receives the state before the chunk.
+// A block owns DC_COLS columns of one head's S for one sequence.  S lies in shared memory, twice (the state before and
+// behind the present chunk); M^T and N of the next chunks are on their way while the present one is multiplied (several
+// chunks ahead where shared memory allows).  A tile of 4 x 4 outputs belongs to PARTS neighbouring lanes, of which lane
+// `part` takes the inner channels part, part + PARTS, ...; their shares are exchanged by shuffles in halves (every lane ends
+// with 16 / PARTS of the outputs), so a chunk takes one barrier.  N's place receives the state before the chunk.
+template <int PARTS>
 __global__ void __launch_bounds__(DC_THREADS)
 delta_walk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     extern __shared__ __align__(16) float sm[];
@@ -282,70 +291,132 @@ delta_walk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     const int hd = blockIdx.x, b = blockIdx.z, tid = threadIdx.x, j0 = blockIdx.y * DC_COLS;
     const int s0 = a.seq_start[b], rows = a.seq_start[b + 1] - s0;
     if (rows <= 0) return;
-    const int D = a.D, DV = a.DV, D4 = g.D4, DV4 = g.DV4, chunks = (rows + DC - 1) / DC;
-    float* Ms = sm;                                     // [2][D4][D4]
-    float* Ns = Ms + 2 * (size_t)D4 * D4;               // [2][D4][DC_COLS]
-    float* S = Ns + 2 * (size_t)D4 * DC_COLS;           // [D4][DC_COLS]
-    float* sh = S + (size_t)D4 * DC_COLS;               // [parts][D4 DC_COLS]
+    const int D = a.D, DV = a.DV, D4 = g.D4, DV4 = g.DV4, ldm = D4 + 4, chunks = (rows + DC - 1) / DC, stages = g.stages;
+    const int m_floats = D4 * ldm, n_floats = D4 * DC_COLS;
+    float* Ms = sm;                                     // [stages][D4][ldm]
+    float* Ns = Ms + stages * (size_t)m_floats;         // [stages][D4][DC_COLS]
+    float* S = Ns + stages * (size_t)n_floats;          // [2][D4][DC_COLS]
     float* st = a.state + (long long)a.seq_slot[b] * a.state_stride + (long long)hd * D * DV;
-    auto fetch = [&](int c) {
-        const float* M = delta_chunk_at(a, g, b, hd, c);
-        const float* N = M + (size_t)D4 * D4;
-        float* md = Ms + (size_t)(c & 1) * D4 * D4;
-        float* nd = Ns + (size_t)(c & 1) * D4 * DC_COLS;
-        for (int e = tid; e < D4 * D4 / 4; e += DC_THREADS) dc_copy16(md + 4 * e, M + 4 * e);
-        for (int e = tid; e < D4 * (DC_COLS / 4); e += DC_THREADS) {
-            const int i = e / (DC_COLS / 4), j = 4 * (e - i * (DC_COLS / 4));
-            if (j0 + j < DV4) dc_copy16(nd + i * DC_COLS + j, N + (size_t)i * DV4 + j0 + j);
+    float* chunk = delta_chunk_at(a, g, b, hd, 0);
+    const int quads = D4 / 4;
+    auto fetch = [&](int c, int slot) {                 // one group of copies per call, empty past the last chunk
+        if (c < chunks) {
+            const float* M = chunk + c * g.stride;
+            const float* N = M + (size_t)D4 * D4;
+            float* md = Ms + (size_t)slot * m_floats;
+            float* nd = Ns + (size_t)slot * n_floats;
+            for (int k = tid >> 4; k < D4; k += DC_THREADS / 16)
+                for (int x = tid & 15; x < quads; x += 16) dc_copy16(md + k * ldm + 4 * x, M + k * D4 + 4 * x);
+            for (int e = tid; e < D4 * (DC_COLS / 4); e += DC_THREADS) {
+                const int i = e / (DC_COLS / 4), j = 4 * (e % (DC_COLS / 4));
+                if (j0 + j < DV4) dc_copy16(nd + i * DC_COLS + j, N + (size_t)i * DV4 + j0 + j);
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0);
-    for (int e = tid; e < D4 * DC_COLS; e += DC_THREADS) {
-        const int i = e / DC_COLS, j = j0 + e - i * DC_COLS;
+    for (int c = 0; c + 1 < stages; ++c) fetch(c, c);
+    for (int e = tid; e < n_floats; e += DC_THREADS) {
+        const int i = e / DC_COLS, j = j0 + e % DC_COLS;
         S[e] = i < D && j < DV ? st[(long long)i * DV + j] : 0.f;
     }
-    for (int e = tid; e < 2 * D4 * DC_COLS; e += DC_THREADS)             // columns past DV4 are never fetched
+    for (int e = tid; e < stages * n_floats; e += DC_THREADS)            // columns past DV4 are never fetched
         if (j0 + e % DC_COLS >= DV4) Ns[e] = 0.f;
     constexpr int CT = DC_COLS / 4;                     // column tiles
-    const int tiles = (D4 / 4) * CT, parts = max(1, DC_THREADS / tiles), share = (D4 + parts - 1) / parts;
+    constexpr int OWN = PARTS >= 16 ? 1 : 16 / PARTS;   // outputs of the tile that a lane ends with
+    const int part = tid % PARTS, tile = tid / PARTS, i0 = 4 * (tile / CT), jt = 4 * (tile % CT);
+    const bool mine = tile < quads * CT;
+    const unsigned everyone = 0xffffffffu;
+    // which outputs (4 x row + column within the tile) the halving leaves with this lane: the first exchange decides the
+    // highest bit
+    int own = 0;
+#pragma unroll
+    for (int o = PARTS / 2, half = 8; o > 0 && half > 0; o >>= 1, half >>= 1) own += (part & o) ? half : 0;
+    const bool writer = mine && (PARTS < 32 || !(part & 1));
+    int slot = 0;
     for (int c = 0; c < chunks; ++c) {
-        if (c + 1 < chunks) {
-            fetch(c + 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();                                // chunk c is here, S is complete
-        const float* M = Ms + (size_t)(c & 1) * D4 * D4;
-        const float* N = Ns + (size_t)(c & 1) * D4 * DC_COLS;
-        float* before = delta_chunk_at(a, g, b, hd, c) + (size_t)D4 * D4;
-        for (int w = tid; w < tiles * parts; w += DC_THREADS) {
-            const int part = w / tiles, tile = w - part * tiles, i = 4 * (tile / CT), j = 4 * (tile % CT);
+        if (stages == 4) asm volatile("cp.async.wait_group 2;" ::: "memory");
+        else if (stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                // chunk c is here, S is complete, the slot of the chunk before is free
+        fetch(c + stages - 1, slot == 0 ? stages - 1 : slot - 1);
+        const float* M = Ms + (size_t)slot * m_floats;
+        const float* N = Ns + (size_t)slot * n_floats;
+        const float* Sb = S + (c & 1) * n_floats;
+        float* Sa = S + ((c + 1) & 1) * n_floats;
+        float v[16];
+        {
             float acc[4][4];
             tile_zero(acc);
-            tile_mac(acc, M + i, D4, S + j, DC_COLS, part * share, min(D4, (part + 1) * share));
-            float* o = sh + (size_t)part * D4 * DC_COLS;
+            if (mine) {
+#pragma unroll 4
+                for (int k = part; k < D4; k += PARTS) {
+                    const float4 x = *reinterpret_cast<const float4*>(M + k * ldm + i0), y = *reinterpret_cast<const float4*>(Sb + k * DC_COLS + jt);
+                    const float xs[4] = {x.x, x.y, x.z, x.w}, ys[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
-            for (int u = 0; u < 4; ++u) *reinterpret_cast<float4*>(o + (i + u) * DC_COLS + j) = make_float4(acc[u][0], acc[u][1], acc[u][2], acc[u][3]);
+                    for (int i = 0; i < 4; ++i)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xs[i], ys[j], acc[i][j]);
+                }
+            }
+#pragma unroll
+            for (int e = 0; e < 16; ++e) v[e] = acc[e >> 2][e & 3];
         }
-        __syncthreads();
-        for (int e = tid; e < D4 * DC_COLS; e += DC_THREADS) {
-            const int i = e / DC_COLS, j = e - i * DC_COLS;
-            float v = N[e];
-            for (int p = 0; p < parts; ++p) v += sh[(size_t)p * D4 * DC_COLS + e];
-            if (j0 + j < DV4) before[(size_t)i * DV4 + j0 + j] = S[e];
-            S[e] = v;
+#pragma unroll
+        for (int o = PARTS / 2, half = 8; o > 0; o >>= 1, half >>= 1) {
+            const bool up = part & o;
+            if (half > 0) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    if (e >= half) break;
+                    const float give = up ? v[e] : v[e + half], keep = up ? v[e + half] : v[e];
+                    v[e] = keep + __shfl_xor_sync(everyone, give, o);
+                }
+            } else {
+                v[0] += __shfl_xor_sync(everyone, v[0], o);
+            }
         }
-        __syncthreads();                                // this chunk's buffers are read: the fetch after the next one takes them
+        if (writer) {
+            float* before = chunk + c * g.stride + (size_t)D4 * D4;
+#pragma unroll
+            for (int e = 0; e < OWN; ++e) {
+                const int out = own + e, i = i0 + (out >> 2), j = jt + (out & 3), at = i * DC_COLS + j;
+                if (j0 + j < DV4) before[(size_t)i * DV4 + j0 + j] = Sb[at];
+                Sa[at] = v[e] + N[at];
+            }
+        }
+        slot = slot + 1 == stages ? 0 : slot + 1;
     }
-    for (int e = tid; e < D4 * DC_COLS; e += DC_THREADS) {
-        const int i = e / DC_COLS, j = j0 + e - i * DC_COLS;
-        if (i < D && j < DV) st[(long long)i * DV + j] = S[e];
+    __syncthreads();
+    const float* Se = S + (chunks & 1) * n_floats;
+    for (int e = tid; e < n_floats; e += DC_THREADS) {
+        const int i = e / DC_COLS, j = j0 + e % DC_COLS;
+        if (i < D && j < DV) st[(long long)i * DV + j] = Se[e];
     }
 }
 
 // ------------------------------------------------------------------------------ pass 3
+// four elements from p on as floats, of which `left` exist (zeros behind them); `vec`: one access
+__device__ __forceinline__ void load_four(float* out, const float* p, int left, bool vec) {
+    if (vec && left > 0) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        out[0] = t.x; out[1] = t.y; out[2] = t.z; out[3] = t.w;
+    } else {
+#pragma unroll
+        for (int v = 0; v < 4; ++v) out[v] = v < left ? p[v] : 0.f;
+    }
+}
+__device__ __forceinline__ void load_four(float* out, const bf16* p, int left, bool vec) {
+    if (vec && left > 0) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        const float2 x = __bfloat1622float2(h[0]), y = __bfloat1622float2(h[1]);
+        out[0] = x.x; out[1] = x.y; out[2] = y.x; out[3] = y.y;
+    } else {
+#pragma unroll
+        for (int v = 0; v < 4; ++v) out[v] = v < left ? __bfloat162float(p[v]) : 0.f;
+    }
+}
+
 // A block takes the 64 rows of a chunk of one head: o = O + Q' S, then the unit norm over the head's channels, the channel
 // weights and the gate's silu.  NT pieces of 64 columns; the sixteen threads of a row's columns are half a warp.
 template <typename T, int NT>
@@ -367,6 +438,9 @@ delta_read_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
         const int i = e / (DC / 4), x = 4 * (e - i * (DC / 4));
         *reinterpret_cast<float4*>(Qs + (size_t)i * DC_LD + x) = *reinterpret_cast<const float4*>(QT + (size_t)i * DC + x);
     }
+    // four neighbouring channels as one access: every head, pitch and base a multiple of four elements
+    const bool vec = DV % 4 == 0 && a.ldp % 4 == 0 && a.ldo % 4 == 0 && (2 * a.G * a.D) % 4 == 0 &&
+                     (((uintptr_t)a.proj | (uintptr_t)a.out) & (4 * sizeof(T) - 1)) == 0 && (((uintptr_t)a.raw | (uintptr_t)a.norm_w) & 15) == 0;
     float o[NT][4][4];
     float ss[4] = {0.f, 0.f, 0.f, 0.f};
     const long long ldr = (long long)H * DV;
@@ -379,16 +453,14 @@ delta_read_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
                 j < DV4 ? *reinterpret_cast<const float4*>(S + (size_t)i * DV4 + j) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
         __syncthreads();
-        tile_zero(o[p]);
+        const int j0 = 64 * p + 4 * tx;
+#pragma unroll
+        for (int u = 0; u < 4; ++u) load_four(o[p][u], a.raw + (r0 + t + u) * ldr + (long long)hd * DV + j0, t + u < n ? DV - j0 : 0, vec);
         tile_mac(o[p], Qs + t, DC_LD, Ss + 4 * tx, DC_LD, 0, D4);
 #pragma unroll
         for (int u = 0; u < 4; ++u)
 #pragma unroll
-            for (int v = 0; v < 4; ++v) {
-                const int j = 64 * p + 4 * tx + v;
-                o[p][u][v] = t + u < n && j < DV ? o[p][u][v] + a.raw[(r0 + t + u) * ldr + (long long)hd * DV + j] : 0.f;
-                ss[u] = fmaf(o[p][u][v], o[p][u][v], ss[u]);
-            }
+            for (int v = 0; v < 4; ++v) ss[u] = fmaf(o[p][u][v], o[p][u][v], ss[u]);
     }
     const int C = 2 * a.G * a.D + H * DV;
 #pragma unroll
@@ -400,14 +472,28 @@ delta_read_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
         const T* G = (const T*)a.proj + (r0 + t + u) * a.ldp + C + (long long)hd * DV;
         T* O = (T*)a.out + (r0 + t + u) * a.ldo + (long long)hd * DV;
 #pragma unroll
-        for (int p = 0; p < NT; ++p)
+        for (int p = 0; p < NT; ++p) {
+            const int j0 = 64 * p + 4 * tx;
+            float gz[4], w[4], y[4];
+            load_four(gz, G + j0, DV - j0, vec);
+            load_four(w, a.norm_w + hd * DV + j0, DV - j0, vec);
 #pragma unroll
-            for (int v = 0; v < 4; ++v) {
-                const int j = 64 * p + 4 * tx + v;
-                if (j >= DV) continue;
-                const float gz = to_f32(G[j]);
-                O[j] = from_f32<T>(((o[p][u][v] * inv) * a.norm_w[hd * DV + j]) * (gz * sigmoid_f32(gz)));
+            for (int v = 0; v < 4; ++v) y[v] = ((o[p][u][v] * inv) * w[v]) * (gz[v] * sigmoid_f32(gz[v]));
+            if (vec && j0 < DV) {
+                if constexpr (sizeof(T) == 2) {
+                    uint2 raw;
+                    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+                    h[0] = __floats2bfloat162_rn(y[0], y[1]);
+                    h[1] = __floats2bfloat162_rn(y[2], y[3]);
+                    *reinterpret_cast<uint2*>(O + j0) = raw;
+                } else {
+                    *reinterpret_cast<float4*>(O + j0) = make_float4(y[0], y[1], y[2], y[3]);
+                }
+            } else {
+                for (int v = 0; v < 4; ++v)
+                    if (j0 + v < DV) O[j0 + v] = from_f32<T>(y[v]);
             }
+        }
     }
 }
 
@@ -424,14 +510,17 @@ int delta_chunked(const DeltaArgs& a, cudaStream_t st) {
     const DeltaChunkGeom g = delta_chunk_geom(a.D, a.DV, a.max_len);
     if (cm_delta_chunk_floats(a.B, a.max_len, a.H, a.D, a.DV) <= 0) CM_REFUSE("delta_chunked: heads of %d x %d", a.D, a.DV);
     const size_t s1 = delta_chunk_smem(g), s2 = delta_walk_smem(g), s3 = delta_read_smem(g);
+    // lanes per tile of pass 2: as many as the block's threads give every tile (64 tiles at most)
+    const int tiles = g.D4 / 4 * (DC_COLS / 4);
+    auto walk = tiles <= 8 ? delta_walk_kernel<32> : tiles <= 16 ? delta_walk_kernel<16> : tiles <= 32 ? delta_walk_kernel<8> : delta_walk_kernel<4>;
     if (cudaFuncSetAttribute(delta_chunk_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess ||
-        cudaFuncSetAttribute(delta_walk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2) != cudaSuccess) {
+        cudaFuncSetAttribute(walk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2) != cudaSuccess) {
         cudaGetLastError();
         CM_REFUSE("delta_chunked: %zu and %zu bytes of shared memory refused", s1, s2);
     }
     cm_launch(delta_chunk_kernel<T>, dim3(g.chunks, a.H, a.B), DC_THREADS, s1, st, a, g);
     CM_CHECK_LAUNCH();
-    cm_launch(delta_walk_kernel, dim3(a.H, (a.DV + DC_COLS - 1) / DC_COLS, a.B), DC_THREADS, s2, st, a, g);
+    cm_launch(walk, dim3(a.H, (a.DV + DC_COLS - 1) / DC_COLS, a.B), DC_THREADS, s2, st, a, g);
     CM_CHECK_LAUNCH();
 #define DC_READ(NT)                                                                                                       \
     do {                                                                                                                  \

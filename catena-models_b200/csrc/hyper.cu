@@ -29,16 +29,14 @@ struct HyperArgs {
 template <typename T, int VEC>
 __device__ __forceinline__ void load_cols(const void* p, bool f32, long long i, float* out) {
     if constexpr (VEC == 4) {
-        if (f32) {
+        if (f32 || sizeof(T) == 4) {
             const float4 t = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
             out[0] = t.x; out[1] = t.y; out[2] = t.z; out[3] = t.w;
-        } else if constexpr (sizeof(T) == 2) {
+        } else {
             const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p) + i);
             const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
             const float2 a = __bfloat1622float2(h[0]), b = __bfloat1622float2(h[1]);
             out[0] = a.x; out[1] = a.y; out[2] = b.x; out[3] = b.y;
-        } else {
-            load_cols<T, VEC>(p, true, i, out);
         }
     } else {
         out[0] = f32 ? reinterpret_cast<const float*>(p)[i] : to_f32(reinterpret_cast<const T*>(p)[i]);

@@ -120,6 +120,46 @@ __device__ void choose_experts(float* sc, float* ch, int E, int top, const Route
         for (int j = 0; j < top; ++j) wts[j] *= r.scale;
 }
 
+// A warp's dot product of two rows of W elements in float (every lane gets it): eight columns a lane and round, where the rows
+// allow 16-byte accesses.
+template <typename T>
+__device__ __forceinline__ float row_dot(const T* __restrict__ w, const T* __restrict__ h, int W, bool vec8) {
+    const int lane = threadIdx.x & 31;
+    float acc = 0.f;
+    if (vec8) {
+#pragma unroll 4
+        for (int c = lane * 8; c < W; c += 256) {
+            float a[8], b[8];
+            load8f<T>(w + c, a);
+            load8f<T>(h + c, b);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc = fmaf(a[i], b[i], acc);
+        }
+    } else {
+        for (int c = lane; c < W; c += 32) acc = fmaf(to_f32(w[c]), to_f32(h[c]), acc);
+    }
+    return warp_sum(acc);
+}
+template <typename T>
+__device__ __forceinline__ bool rows_vec8(const T* a, const T* b, int W) {
+    return W % 8 == 0 && ((((uintptr_t)a) | ((uintptr_t)b)) & 15) == 0;
+}
+// dst = T(src * w) for one row, threads `at`, at + step, ...
+template <typename T>
+__device__ __forceinline__ void copy_scaled(T* __restrict__ dst, const T* __restrict__ src, float w, int W, int at, int step) {
+    if (rows_vec8(dst, src, W)) {
+        for (int c = at * 8; c < W; c += step * 8) {
+            float x[8];
+            load8f<T>(src + c, x);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[i] *= w;
+            store8f<T>(dst + c, x);
+        }
+    } else {
+        for (int c = at; c < W; c += step) dst[c] = from_f32<T>(to_f32(src[c]) * w);
+    }
+}
+
 // One block per token.  ids[p] = expert of pair p (-1 for rows of padding), wts[p] its weight.
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -136,11 +176,9 @@ moe_router_kernel(int* __restrict__ ids, float* __restrict__ wts, int* __restric
     }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const T* hr = h + t * W;
+    const bool vec8 = rows_vec8(h, wr, W);
     for (int e = warp; e < E; e += 4) {
-        const T* w = wr + (long long)e * W;
-        float acc = 0.f;
-        for (int c = lane; c < W; c += 32) acc = fmaf(to_f32(w[c]), to_f32(hr[c]), acc);
-        acc = warp_sum(acc);
+        const float acc = row_dot<T>(wr + (long long)e * W, hr, W, vec8);
         if (lane == 0) score[e] = acc;
     }
     __syncthreads();
@@ -200,9 +238,7 @@ __global__ void moe_gather_kernel(T* __restrict__ xs, const T* __restrict__ h, c
     const int d = dest[p];
     if (d < 0) return;
     const float w = apply_weight ? wts[p] : 1.f;
-    const T* src = h + (p / top) * K;
-    T* dst = xs + (long long)d * K;
-    for (int c = threadIdx.x; c < K; c += blockDim.x) dst[c] = from_f32<T>(to_f32(src[c]) * w);
+    copy_scaled<T>(xs + (long long)d * K, h + (p / top) * K, w, K, threadIdx.x, blockDim.x);
 }
 
 extern "C" int cm_moe_gather(int dt, void* xs, const void* h, const int* dest, const float* wts, long long pairs,
@@ -221,9 +257,10 @@ extern "C" int cm_moe_gather(int dt, void* xs, const void* h, const int* dest, c
 // Everything above in one block, for the few rows of a decode step: scores, the best `top`, counts, the list of
 // row tiles, the order of the pairs, and (with xs) the experts' inputs in that order.  One launch instead of five.
 #define MOE_SMALL_ROWS 64
+#define MOE_SMALL_THREADS 512
 #define MOE_SMALL_SCORES 8192
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(MOE_SMALL_THREADS)
 moe_route_small_kernel(int* __restrict__ ids, float* __restrict__ wts, int* __restrict__ perm, int* __restrict__ dest,
                        int* __restrict__ counts_out, int* __restrict__ plan, int* __restrict__ tile_group,
                        const T* __restrict__ h, const T* __restrict__ wr, const int* __restrict__ tok_seq, int rows, int W,
@@ -238,13 +275,10 @@ moe_route_small_kernel(int* __restrict__ ids, float* __restrict__ wts, int* __re
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
-    for (int pe = warp; pe < rows * E; pe += 8) {
+    const bool vec8 = rows_vec8(h, wr, W);
+    for (int pe = warp; pe < rows * E; pe += MOE_SMALL_THREADS / 32) {
         const int t = pe / E, e = pe - t * E;
-        const T* w = wr + (long long)e * W;
-        const T* hr = h + (long long)t * W;
-        float acc = 0.f;
-        for (int c = lane; c < W; c += 32) acc = fmaf(to_f32(w[c]), to_f32(hr[c]), acc);
-        acc = warp_sum(acc);
+        const float acc = row_dot<T>(wr + (long long)e * W, h + (long long)t * W, W, vec8);
         if (lane == 0) score[pe] = acc;
     }
     __syncthreads();
@@ -287,13 +321,10 @@ moe_route_small_kernel(int* __restrict__ ids, float* __restrict__ wts, int* __re
     }
     if (!xs) return;
     __syncthreads();                              // dest and wts of this block's own writes
-    for (int p = warp; p < P; p += 8) {
+    for (int p = warp; p < P; p += MOE_SMALL_THREADS / 32) {
         const int d = dest[p];
         if (d < 0) continue;
-        const float w = apply_weight ? wts[p] : 1.f;
-        const T* src = h + (long long)(p / top) * W;
-        T* dst = xs + (long long)d * W;
-        for (int c = lane; c < W; c += 32) dst[c] = from_f32<T>(to_f32(src[c]) * w);
+        copy_scaled<T>(xs + (long long)d * W, h + (long long)(p / top) * W, apply_weight ? wts[p] : 1.f, W, lane, 32);
     }
 }
 
@@ -343,11 +374,11 @@ extern "C" int cm_moe_route(int dt, int* ids, float* wts, int* perm, int* dest, 
     if (rows <= MOE_SMALL_ROWS && rows * E * (two ? 2 : 1) <= MOE_SMALL_SCORES && (dt == DT_F32 || dt == DT_BF16)) {
         const size_t small = ((size_t)rows * E * (two ? 2 : 1)) * sizeof(float) + 2 * (size_t)E * sizeof(int);
         if (dt == DT_F32)
-            cm_launch(moe_route_small_kernel<float>, 1, 256, small, st, ids, wts, perm, dest, counts, plan, tile_group,
+            cm_launch(moe_route_small_kernel<float>, 1, MOE_SMALL_THREADS, small, st, ids, wts, perm, dest, counts, plan, tile_group,
                       (const float*)h, (const float*)wr, tok_seq, (int)rows, W, E, top, rule, tile_rows,
                       max_tiles, (float*)xs, apply_weight);
         else
-            cm_launch(moe_route_small_kernel<bf16>, 1, 256, small, st, ids, wts, perm, dest, counts, plan, tile_group,
+            cm_launch(moe_route_small_kernel<bf16>, 1, MOE_SMALL_THREADS, small, st, ids, wts, perm, dest, counts, plan, tile_group,
                       (const bf16*)h, (const bf16*)wr, tok_seq, (int)rows, W, E, top, rule, tile_rows,
                       max_tiles, (bf16*)xs, apply_weight);
         CM_CHECK_LAUNCH();

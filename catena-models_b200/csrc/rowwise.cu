@@ -446,6 +446,7 @@ extern "C" int cm_scale_softcap(float* x, long long total, float scale, float ca
 }
 
 // ----------------------------------------------------------------------- row gather
+#define GATHER_COLS 1024
 template <typename T>
 __global__ void gather_rows_kernel(T* __restrict__ out, const T* __restrict__ x,
                                    const int* __restrict__ rows, int H) {
@@ -453,16 +454,22 @@ __global__ void gather_rows_kernel(T* __restrict__ out, const T* __restrict__ x,
     pdl_wait();
     const T* src = x + (long long)rows[blockIdx.x] * H;
     T* dst = out + (long long)blockIdx.x * H;
-    for (int c = threadIdx.x; c < H; c += blockDim.x) dst[c] = src[c];
+    const int c0 = blockIdx.y * GATHER_COLS;           // a row's columns are dealt to blocks: few rows are wanted, wide ones
+#pragma unroll
+    for (int u = 0; u < GATHER_COLS / 128; ++u) {
+        const int c = c0 + u * 128 + threadIdx.x;
+        if (c < H) dst[c] = src[c];
+    }
 }
 
 extern "C" int cm_gather_rows(int dt, void* out, const void* x, const int* rows, int n, int H,
                               cudaStream_t st) {
-    if (n <= 0) return CM_OK;
+    if (n <= 0 || H <= 0) return CM_OK;
+    const dim3 grid(n, (H + GATHER_COLS - 1) / GATHER_COLS);
     if (dt == DT_F32)
-        cm_launch(gather_rows_kernel<float>, n, 128, 0, st, (float*)out, (const float*)x, rows, H);
+        cm_launch(gather_rows_kernel<float>, grid, 128, 0, st, (float*)out, (const float*)x, rows, H);
     else if (dt == DT_BF16)
-        cm_launch(gather_rows_kernel<bf16>, n, 128, 0, st, (bf16*)out, (const bf16*)x, rows, H);
+        cm_launch(gather_rows_kernel<bf16>, grid, 128, 0, st, (bf16*)out, (const bf16*)x, rows, H);
     else
         return CM_ERR_DTYPE;
     CM_CHECK_LAUNCH();
