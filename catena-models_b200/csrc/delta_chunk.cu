@@ -32,13 +32,14 @@ struct DeltaChunkGeom {
     long long stride;            // floats of one chunk of one head in the scratch: M^T [D4][D4], N [D4][DV4], Q'^T [D4][DC]
 };
 
+static __host__ __device__ __forceinline__ constexpr int dc_stages(int D4) { return D4 <= 64 ? 4 : (D4 <= 96 ? 3 : 2); }
 static __host__ __device__ __forceinline__ DeltaChunkGeom delta_chunk_geom(int D, int DV, int max_len) {
     DeltaChunkGeom g;
     g.D4 = (D + 3) & ~3;
     g.DV4 = (DV + 3) & ~3;
     g.chunks = (max_len + DC - 1) / DC;
     g.NCp = g.D4 + g.DV4 + 4;
-    g.stages = g.D4 <= 64 ? 4 : (g.D4 <= 96 ? 3 : 2);
+    g.stages = dc_stages(g.D4);
     g.stride = (long long)g.D4 * (g.D4 + g.DV4 + DC);
     return g;
 }
@@ -81,7 +82,8 @@ __device__ __forceinline__ void tile_zero(float (&acc)[4][4]) {
 }
 
 // ------------------------------------------------------------------------------ pass 1
-template <typename T>
+// DK, DVK: the heads' sizes where they are known to the compiler (multiples of 4), or 0.
+template <typename T, int DK, int DVK>
 __global__ void __launch_bounds__(DC_THREADS, 2)
 delta_chunk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     extern __shared__ __align__(16) float sm[];
@@ -92,7 +94,8 @@ delta_chunk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     const long long r0 = (long long)s0 + (long long)c * DC;
     const int n = (int)min((long long)DC, s1 - r0);
     if (n <= 0) return;
-    const int D = a.D, DV = a.DV, H = a.H, G = a.G, kh = hd / (H / G), D4 = g.D4, DV4 = g.DV4, NC = D4 + DV4, NCp = g.NCp, ldk = D4 + 4;
+    const int D = DK ? DK : a.D, DV = DVK ? DVK : a.DV, D4 = DK ? DK : g.D4, DV4 = DVK ? DVK : g.DV4;
+    const int H = a.H, G = a.G, kh = hd / (H / G), NC = D4 + DV4, NCp = NC + 4, ldk = D4 + 4;
     const size_t first = 2 * (size_t)D4 * DC_LD, xsz = (size_t)DC * NCp;
     float* kT = sm;                                     // [D4][DC_LD]: k_t,i at [i][t]
     float* qT = kT + (size_t)D4 * DC_LD;                // the same of q
@@ -282,7 +285,7 @@ __device__ __forceinline__ void dc_copy16(float* dst, const float* src) {
 // chunks ahead where shared memory allows).  A tile of 4 x 4 outputs belongs to PARTS neighbouring lanes, of which lane
 // `part` takes the inner channels part, part + PARTS, ...; their shares are exchanged by shuffles in halves (every lane ends
 // with 16 / PARTS of the outputs), so a chunk takes one barrier.  N's place receives the state before the chunk.
-template <int PARTS>
+template <int PARTS, int DK>
 __global__ void __launch_bounds__(DC_THREADS)
 delta_walk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     extern __shared__ __align__(16) float sm[];
@@ -291,7 +294,8 @@ delta_walk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     const int hd = blockIdx.x, b = blockIdx.z, tid = threadIdx.x, j0 = blockIdx.y * DC_COLS;
     const int s0 = a.seq_start[b], rows = a.seq_start[b + 1] - s0;
     if (rows <= 0) return;
-    const int D = a.D, DV = a.DV, D4 = g.D4, DV4 = g.DV4, ldm = D4 + 4, chunks = (rows + DC - 1) / DC, stages = g.stages;
+    const int D = DK ? DK : a.D, DV = a.DV, D4 = DK ? DK : g.D4, DV4 = g.DV4, ldm = D4 + 4, chunks = (rows + DC - 1) / DC;
+    const int stages = DK ? dc_stages(DK) : g.stages;
     const int m_floats = D4 * ldm, n_floats = D4 * DC_COLS;
     float* Ms = sm;                                     // [stages][D4][ldm]
     float* Ns = Ms + stages * (size_t)m_floats;         // [stages][D4][DC_COLS]
@@ -419,7 +423,7 @@ __device__ __forceinline__ void load_four(float* out, const bf16* p, int left, b
 
 // A block takes the 64 rows of a chunk of one head: o = O + Q' S, then the unit norm over the head's channels, the channel
 // weights and the gate's silu.  NT pieces of 64 columns; the sixteen threads of a row's columns are half a warp.
-template <typename T, int NT>
+template <typename T, int NT, int DK>
 __global__ void __launch_bounds__(DC_THREADS)
 delta_read_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     extern __shared__ __align__(16) float sm[];
@@ -429,7 +433,7 @@ delta_read_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     const long long r0 = (long long)a.seq_start[b] + (long long)c * DC;
     const int n = (int)min((long long)DC, a.seq_start[b + 1] - r0);
     if (n <= 0) return;
-    const int DV = a.DV, D4 = g.D4, DV4 = g.DV4, H = a.H, ty = tid >> 4, tx = tid & 15, t = 4 * ty;
+    const int DV = a.DV, D4 = DK ? DK : g.D4, DV4 = g.DV4, H = a.H, ty = tid >> 4, tx = tid & 15, t = 4 * ty;
     float* Qs = sm;                                     // [D4][DC_LD]: Q'^T
     float* Ss = Qs + (size_t)D4 * DC_LD;                // [D4][DC_LD]: 64 columns of the state before the chunk
     const float* S = delta_chunk_at(a, g, b, hd, c) + (size_t)D4 * D4;
@@ -512,26 +516,44 @@ int delta_chunked(const DeltaArgs& a, cudaStream_t st) {
     const size_t s1 = delta_chunk_smem(g), s2 = delta_walk_smem(g), s3 = delta_read_smem(g);
     // lanes per tile of pass 2: as many as the block's threads give every tile (64 tiles at most)
     const int tiles = g.D4 / 4 * (DC_COLS / 4);
-    auto walk = tiles <= 8 ? delta_walk_kernel<32> : tiles <= 16 ? delta_walk_kernel<16> : tiles <= 32 ? delta_walk_kernel<8> : delta_walk_kernel<4>;
-    if (cudaFuncSetAttribute(delta_chunk_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess ||
+    auto walk = a.D == 64    ? delta_walk_kernel<8, 64>
+                : a.D == 128 ? delta_walk_kernel<4, 128>
+                : tiles <= 8 ? delta_walk_kernel<32, 0>
+                : tiles <= 16 ? delta_walk_kernel<16, 0>
+                : tiles <= 32 ? delta_walk_kernel<8, 0>
+                              : delta_walk_kernel<4, 0>;
+    auto first = delta_chunk_kernel<T, 0, 0>;
+    if constexpr (sizeof(T) == 2) {
+        if (a.D == 64 && a.DV == 64) first = delta_chunk_kernel<T, 64, 64>;
+        else if (a.D == 64 && a.DV == 128) first = delta_chunk_kernel<T, 64, 128>;
+        else if (a.D == 128 && a.DV == 128) first = delta_chunk_kernel<T, 128, 128>;
+    }
+    if (cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess ||
         cudaFuncSetAttribute(walk, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2) != cudaSuccess) {
         cudaGetLastError();
         CM_REFUSE("delta_chunked: %zu and %zu bytes of shared memory refused", s1, s2);
     }
-    cm_launch(delta_chunk_kernel<T>, dim3(g.chunks, a.H, a.B), DC_THREADS, s1, st, a, g);
+    cm_launch(first, dim3(g.chunks, a.H, a.B), DC_THREADS, s1, st, a, g);
     CM_CHECK_LAUNCH();
     cm_launch(walk, dim3(a.H, (a.DV + DC_COLS - 1) / DC_COLS, a.B), DC_THREADS, s2, st, a, g);
     CM_CHECK_LAUNCH();
-#define DC_READ(NT)                                                                                                       \
+#define DC_READ(NT)                          \
+    do {                                     \
+        if (a.D == 64) DC_READ_D(NT, 64);    \
+        else if (a.D == 128) DC_READ_D(NT, 128); \
+        else DC_READ_D(NT, 0);               \
+    } while (0)
+#define DC_READ_D(NT, DK)                                                                                                       \
     do {                                                                                                                  \
-        cudaFuncSetAttribute(delta_read_kernel<T, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);             \
-        cm_launch(delta_read_kernel<T, NT>, dim3(g.chunks, a.H, a.B), DC_THREADS, s3, st, a, g);                          \
+        cudaFuncSetAttribute(delta_read_kernel<T, NT, DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);             \
+        cm_launch(delta_read_kernel<T, NT, DK>, dim3(g.chunks, a.H, a.B), DC_THREADS, s3, st, a, g);                          \
     } while (0)
     if (a.DV <= 64) DC_READ(1);
     else if (a.DV <= 128) DC_READ(2);
     else if (a.DV <= 192) DC_READ(3);
     else DC_READ(4);
 #undef DC_READ
+#undef DC_READ_D
     CM_CHECK_LAUNCH();
     return CM_OK;
 }

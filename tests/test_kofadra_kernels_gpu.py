@@ -256,7 +256,7 @@ def _delta_part(W, H, G, D, DV, taps, eps, dtype, seed):
 @pytest.mark.parametrize("dtype, tol", [(torch.float32, 2e-5), (torch.bfloat16, 3e-2)])
 @pytest.mark.parametrize("W, H, G, D, DV, taps", [
     (32, 4, 2, 16, 24, 4), (24, 1, 1, 8, 8, 1), (40, 3, 3, 7, 9, 2), (64, 4, 1, 64, 128, 3), (48, 2, 1, 128, 64, 4), (32, 2, 2, 4, 36, 5),
-    (40, 2, 1, 20, 132, 4), (32, 1, 1, 150, 40, 3), (32, 2, 1, 96, 200, 16)])
+    (40, 2, 1, 20, 132, 4), (32, 1, 1, 150, 40, 3), (32, 2, 1, 96, 200, 16), (32, 2, 1, 64, 64, 4), (40, 2, 2, 128, 128, 2)])
 def test_delta_rule_whole_portions_single_tokens_and_slots(W, H, G, D, DV, taps, dtype, tol):
     """Three sequences of unequal length, whole, in portions, two tokens at a time and token by token, on slots that were
     used before; head sizes with and without the one-kernel step and the chunked form."""
