@@ -241,7 +241,6 @@ template <typename T, int RPT>
 __global__ void __launch_bounds__(DS_THREADS)
 delta_scan_kernel(const DeltaArgs a, int KS, int TB) {
     extern __shared__ __align__(16) float sm[];
-    pdl_trigger();
     pdl_wait();
     const int hd = blockIdx.x, cb = blockIdx.y, b = blockIdx.z;
     const int s0 = a.seq_start[b], s1 = a.seq_start[b + 1];
@@ -301,17 +300,30 @@ delta_scan_kernel(const DeltaArgs a, int KS, int TB) {
             sg[2 * tt + 1] = a.lb[(t0 + tt) * 2 * H + H + hd];
         }
         __syncthreads();
-#pragma unroll 2
+        // the operands of a row are fetched a row ahead (the shares stored below could alias them for all the compiler knows)
+        float kn[RPT], qn[RPT], gn, bn, vn;
+        auto fetch = [&](int tt) {
+#pragma unroll
+            for (int x = 0; x < RPT / 4; ++x) {
+                const float4 kq = *reinterpret_cast<const float4*>(sk + tt * Dp + 4 * (ks + KS * x));
+                const float4 qq = *reinterpret_cast<const float4*>(sq + tt * Dp + 4 * (ks + KS * x));
+                kn[4 * x] = kq.x; kn[4 * x + 1] = kq.y; kn[4 * x + 2] = kq.z; kn[4 * x + 3] = kq.w;
+                qn[4 * x] = qq.x; qn[4 * x + 1] = qq.y; qn[4 * x + 2] = qq.z; qn[4 * x + 3] = qq.w;
+            }
+            gn = sg[2 * tt];
+            bn = sg[2 * tt + 1];
+            vn = sv[tt * cols + c];
+        };
+        fetch(0);
         for (int tt = 0; tt < nt; ++tt) {
             float q[RPT], k[RPT];
 #pragma unroll
-            for (int x = 0; x < RPT / 4; ++x) {
-                const float4 kq = *reinterpret_cast<const float4*>(sk + (size_t)tt * Dp + 4 * (ks + KS * x));
-                const float4 qq = *reinterpret_cast<const float4*>(sq + (size_t)tt * Dp + 4 * (ks + KS * x));
-                k[4 * x] = kq.x; k[4 * x + 1] = kq.y; k[4 * x + 2] = kq.z; k[4 * x + 3] = kq.w;
-                q[4 * x] = qq.x; q[4 * x + 1] = qq.y; q[4 * x + 2] = qq.z; q[4 * x + 3] = qq.w;
+            for (int it = 0; it < RPT; ++it) {
+                k[it] = kn[it];
+                q[it] = qn[it];
             }
-            const float g = sg[2 * tt], beta = sg[2 * tt + 1], vj = sv[tt * cols + c];
+            const float g = gn, beta = bn, vj = vn;
+            fetch(min(tt + 1, nt - 1));
             float d4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int it = 0; it < RPT; ++it) {
@@ -319,7 +331,9 @@ delta_scan_kernel(const DeltaArgs a, int KS, int TB) {
                 d4[it & 3] = fmaf(S[it], k[it], d4[it & 3]);
             }
             float dot = (d4[0] + d4[1]) + (d4[2] + d4[3]);
-            for (int o = KS >> 1; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+                if (o < KS) dot += __shfl_xor_sync(0xffffffffu, dot, o);
             const float u = beta * (vj - dot);
             float a4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -327,7 +341,7 @@ delta_scan_kernel(const DeltaArgs a, int KS, int TB) {
                 S[it] = fmaf(k[it], u, S[it]);
                 a4[it & 3] = fmaf(S[it], q[it], a4[it & 3]);
             }
-            part[((size_t)tt * KS + ks) * cols + c] = (a4[0] + a4[1]) + (a4[2] + a4[3]);
+            part[(tt * KS + ks) * cols + c] = (a4[0] + a4[1]) + (a4[2] + a4[3]);
         }
         __syncthreads();
         for (int e = threadIdx.x; e < nt * cols; e += DS_THREADS) {
@@ -338,6 +352,7 @@ delta_scan_kernel(const DeltaArgs a, int KS, int TB) {
             R[(t0 + tt) * ldv + cc] = o;
         }
     }
+    pdl_trigger();
 #pragma unroll
     for (int it = 0; it < RPT; ++it) {
         const int i = 4 * (ks + KS * (it >> 2)) + (it & 3);
@@ -360,7 +375,9 @@ static int launch_delta_scan(const DeltaArgs& a, cudaStream_t st) {
     tb = tb < 1 ? 1 : (tb > DS_MAX_ROWS ? DS_MAX_ROWS : tb);
     const size_t smem = (size_t)tb * row_floats * sizeof(float);
     dim3 grid(a.H, (a.DV + cols - 1) / cols, a.B);
-#define DS_LAUNCH(R) cm_launch(delta_scan_kernel<T, R>, grid, DS_THREADS, smem, st, a, ks, tb)
+    // In plain stream order: blocks that start early land on whichever SMs have room while the kernel before drains, several
+    // on one, and stay there for the whole walk (measured on B200, 2,048 rows, 16 heads of 64 x 128: 865 against 575 us).
+#define DS_LAUNCH(R) cm_launch_cluster(delta_scan_kernel<T, R>, grid, DS_THREADS, smem, st, 1, false, a, ks, tb)
     if (rpt == 4) DS_LAUNCH(4);
     else if (rpt == 8) DS_LAUNCH(8);
     else if (rpt == 16) DS_LAUNCH(16);

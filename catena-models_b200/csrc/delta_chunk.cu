@@ -87,7 +87,6 @@ template <typename T, int DK, int DVK>
 __global__ void __launch_bounds__(DC_THREADS, 2)
 delta_chunk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     extern __shared__ __align__(16) float sm[];
-    pdl_trigger();
     pdl_wait();
     const int c = blockIdx.x, hd = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
     const int s0 = a.seq_start[b], s1 = a.seq_start[b + 1];
@@ -221,6 +220,7 @@ delta_chunk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
         kr[(size_t)r * ldk + i] *= de[r];
     }
     __syncthreads();
+    pdl_trigger();                                      // not before: waiting blocks of the next pass would take this one's room
     float* MT = delta_chunk_at(a, g, b, hd, c);
     float* N = MT + (size_t)D4 * D4;
     float* QT = N + (size_t)D4 * DV4;
@@ -289,7 +289,6 @@ template <int PARTS, int DK>
 __global__ void __launch_bounds__(DC_THREADS)
 delta_walk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     extern __shared__ __align__(16) float sm[];
-    pdl_trigger();
     pdl_wait();
     const int hd = blockIdx.x, b = blockIdx.z, tid = threadIdx.x, j0 = blockIdx.y * DC_COLS;
     const int s0 = a.seq_start[b], rows = a.seq_start[b + 1] - s0;
@@ -390,6 +389,7 @@ delta_walk_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
         }
         slot = slot + 1 == stages ? 0 : slot + 1;
     }
+    pdl_trigger();
     __syncthreads();
     const float* Se = S + (chunks & 1) * n_floats;
     for (int e = tid; e < n_floats; e += DC_THREADS) {
@@ -427,7 +427,6 @@ template <typename T, int NT, int DK>
 __global__ void __launch_bounds__(DC_THREADS)
 delta_read_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
     extern __shared__ __align__(16) float sm[];
-    pdl_trigger();
     pdl_wait();
     const int c = blockIdx.x, hd = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
     const long long r0 = (long long)a.seq_start[b] + (long long)c * DC;
@@ -466,6 +465,7 @@ delta_read_kernel(const DeltaArgs a, const DeltaChunkGeom g) {
 #pragma unroll
             for (int v = 0; v < 4; ++v) ss[u] = fmaf(o[p][u][v], o[p][u][v], ss[u]);
     }
+    pdl_trigger();
     const int C = 2 * a.G * a.D + H * DV;
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
@@ -535,7 +535,8 @@ int delta_chunked(const DeltaArgs& a, cudaStream_t st) {
     }
     cm_launch(first, dim3(g.chunks, a.H, a.B), DC_THREADS, s1, st, a, g);
     CM_CHECK_LAUNCH();
-    cm_launch(walk, dim3(a.H, (a.DV + DC_COLS - 1) / DC_COLS, a.B), DC_THREADS, s2, st, a, g);
+    // in plain stream order, so that its blocks spread evenly over the SMs (see launch_delta_scan)
+    cm_launch_cluster(walk, dim3(a.H, (a.DV + DC_COLS - 1) / DC_COLS, a.B), DC_THREADS, s2, st, 1, false, a, g);
     CM_CHECK_LAUNCH();
 #define DC_READ(NT)                          \
     do {                                     \
