@@ -172,8 +172,15 @@ struct FtPast {                      // where the keys and values below a sequen
 struct FtItem {
     int b, hq, hk, s0, len, q0, p0, kt_begin, tp_begin, n_past, n;
 };
-// Item w of the launch, long rows first (the query tile falls as w rises).  n = 0: nothing to do (the
-// sequence is shorter than this tile's first row).
+// Query tiles that a chunk of the mask spans, at most (`tiles_x`: of the longest sequence); 0: the mask does not go by chunks.
+static __host__ __device__ __forceinline__ int ft_chunk_tiles(int window, int tiles_x) {
+    if (window >= 0) return 0;
+    const int t = (-window + FT_TILE - 1) / FT_TILE;
+    return t < tiles_x ? t : tiles_x;
+}
+// Item w of the launch, long rows first: the query tile falls as w rises; under a mask by chunks the last tiles of all
+// chunks come first, then the ones before them, and so on (tiles_x is then a multiple of a chunk's tiles).  n = 0:
+// nothing to do (the sequence is shorter than this tile's first row).
 template <bool PAST>
 __device__ __forceinline__ void ft_item(int w, int tiles_x, int QH, int KVH, int B, int window,
                                         const int* __restrict__ seq_start, const FtPast& past, FtItem& it) {
@@ -183,7 +190,13 @@ __device__ __forceinline__ void ft_item(int w, int tiles_x, int QH, int KVH, int
     it.hk = it.hq / (QH / KVH);
     it.s0 = seq_start[it.b];
     it.len = seq_start[it.b + 1] - it.s0;
-    it.q0 = (tiles_x - 1 - x) * FT_TILE;
+    const int ct = ft_chunk_tiles(window, tiles_x);
+    if (ct > 1) {
+        const int chunks = tiles_x / ct, back = x / chunks;
+        it.q0 = ((x - back * chunks) * ct + ct - 1 - back) * FT_TILE;
+    } else {
+        it.q0 = (tiles_x - 1 - x) * FT_TILE;
+    }
     it.n = 0;
     it.p0 = 0;
     it.kt_begin = it.tp_begin = it.n_past = 0;
@@ -748,7 +761,8 @@ static int launch_ft(void* ctx, long long ldc, const void* q, const void* k, con
         cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev);
         if (sm_count <= 0) sm_count = 1;
     }
-    const int tiles_x = (max_len + FT_TILE - 1) / FT_TILE;
+    int tiles_x = (max_len + FT_TILE - 1) / FT_TILE;
+    if (const int ct = ft_chunk_tiles(window, tiles_x); ct > 1) tiles_x = (tiles_x + ct - 1) / ct * ct;      // whole chunks: see ft_item
     const long long items = (long long)tiles_x * QH * B;
     if (items > 0x7fffffffLL) CM_REFUSE("attn_prefill_tc: %lld items", items);
     const long long blocks = SOLO ? (items + 1) / 2 : items;
