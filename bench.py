@@ -793,7 +793,7 @@ def main():
     ap.add_argument("--compare", default=None, choices=["narasun", "fozedra", "maferax", "relilix", "kofadra"],
                     help="instead of the JSON line: prompt and decode throughput of that design beside the closest earlier "
                          "one at equal size (random weights: Narasun beside LFM3, Fozedra and Maferax beside Narasun, Relilix beside "
-                         "Maferax), as a table")
+                         "Maferax, Kofadra beside Narasun and Maferax), as a table")
     ap.add_argument("--compare-sizes", default="1024,2048", help="widths of `--compare`")
     ap.add_argument("--compare-kernels", action="store_true", help="with `--compare`: also each model's kernel tables")
     ap.add_argument("--print-config", action="store_true",
