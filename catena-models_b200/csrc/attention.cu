@@ -1,6 +1,10 @@
 // Attention kernels: head norm + rotation + cache write, prefill attention over the step's
 // own keys, decode attention over the paged cache (split over fixed chunks, ordered merge).
 //
+// What leaves an attention (all forms, also those of attention_mma.cu and attention_tc.cu): the first DV of a head's HD
+// value channels, side by side per row (head h at column h * DV; DV = HD unless heads are padded with zeros), times
+// sigmoid(gate): one logit per head at gate[row][h], or with gate_ch one per channel at gate[row][h * DV + d].
+//
 // Masks: a key at position k is visible to a query at position p when k <= p and k is not before
 // first_visible(p, window): for a window W > 0, k + W > p; for W < 0, k lies in p's chunk of -W
 // positions.  Scores, softmax and the probability-value sums are float.
@@ -322,7 +326,7 @@ attn_prefill_simt_kernel(T* __restrict__ ctx, long long ldc, const T* __restrict
                          const int* __restrict__ seq_start, int QH, int KVH, int HD, int window,
                          float scale, const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot,
                          const T* __restrict__ pool, long long pages, const int* __restrict__ ptab,
-                         int ptab_stride, int ring, const float* __restrict__ sink, float cap) {
+                         int ptab_stride, int ring, const float* __restrict__ sink, float cap, int DV, int gate_ch) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float smem[];
@@ -426,12 +430,14 @@ attn_prefill_simt_kernel(T* __restrict__ ctx, long long ldc, const T* __restrict
         if (qi >= nq) continue;
         const long long t = s0 + q0 - p0 + qi;
         float g = 1.f;
-        if (gate) g = sigmoid_f32(to_f32(gate[t * ldg + hq]));
+        if (gate && !gate_ch) g = sigmoid_f32(to_f32(gate[t * ldg + hq]));
         const float inv = 1.f / (l[i] + (sink ? expf(sink[hq] - m[i]) : 0.f));   // a sink joins the denominator only
 #pragma unroll
         for (int j = 0; j < AP_MAXJ; ++j) {
             const int d = lane + 32 * j;
-            if (j < nj && d < HD) ctx[t * ldc + (long long)hq * HD + d] = from_f32<T>(acc[i][j] * inv * g);
+            if (j >= nj || d >= DV) continue;
+            if (gate && gate_ch) g = sigmoid_f32(to_f32(gate[t * ldg + (long long)hq * DV + d]));
+            ctx[t * ldc + (long long)hq * DV + d] = from_f32<T>(acc[i][j] * inv * g);
         }
     }
 }
@@ -441,13 +447,14 @@ static int launch_attn_simt(void* ctx, long long ldc, const void* q, const void*
                             const void* gate, long long ldg, const int* seq_start, int B, int max_len, int QH, int KVH,
                             int HD, int window, float scale, const int* seq_pos0, const int* seq_slot, const void* pool,
                             long long pages, const int* ptab, int ptab_stride, int ring, const float* sink, float cap,
-                            cudaStream_t st) {
+                            int DV, int gate_ch, cudaStream_t st) {
+    if (DV < 1 || DV > HD) CM_REFUSE("attention: %d of %d channels stored", DV, HD);
     const size_t smem = ((size_t)(AP_BQ + AP_BK) * (HD + 1) + (size_t)AP_BK * HD + AP_BQ * (AP_BK + 1)) * sizeof(float);
     dim3 grid((max_len + AP_BQ - 1) / AP_BQ, QH, B);
     cudaFuncSetAttribute(attn_prefill_simt_kernel<T, PAST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     cm_launch(attn_prefill_simt_kernel<T, PAST>, grid, 128, smem, st, (T*)ctx, ldc, (const T*)q, (const T*)k, (const T*)v,
               ld, (const T*)gate, ldg, seq_start, QH, KVH, HD, window, scale, seq_pos0, seq_slot, (const T*)pool, pages,
-              ptab, ptab_stride, ring, sink, cap);
+              ptab, ptab_stride, ring, sink, cap, DV, gate_ch);
     CM_CHECK_LAUNCH();
     return CM_OK;
 }
@@ -455,16 +462,17 @@ static int launch_attn_simt(void* ctx, long long ldc, const void* q, const void*
 extern "C" int cm_attn_prefill_simt(int dt, void* ctx, long long ldc, const void* q, const void* k,
                                     const void* v, long long ld, const void* gate, long long ldg,
                                     const int* seq_start, int B, int max_len, int QH, int KVH, int HD,
-                                    int window, float scale, float softcap, const float* sink, cudaStream_t st) {
+                                    int window, float scale, float softcap, const float* sink, int DV, int gate_ch,
+                                    cudaStream_t st) {
     if (B <= 0 || max_len <= 0) return CM_OK;
     if (HD > 32 * AP_MAXJ) CM_REFUSE("attn_prefill: head size %d above %d", HD, 32 * AP_MAXJ);
     if (QH % KVH) CM_REFUSE("attn_prefill: %d query heads over %d key heads", QH, KVH);
     if (dt == DT_F32)
         return launch_attn_simt<float, false>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, QH, KVH, HD, window,
-                                              scale, nullptr, nullptr, nullptr, 0, nullptr, 0, 0, sink, softcap, st);
+                                              scale, nullptr, nullptr, nullptr, 0, nullptr, 0, 0, sink, softcap, DV, gate_ch, st);
     if (dt == DT_BF16)
         return launch_attn_simt<bf16, false>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, QH, KVH, HD, window,
-                                             scale, nullptr, nullptr, nullptr, 0, nullptr, 0, 0, sink, softcap, st);
+                                             scale, nullptr, nullptr, nullptr, 0, nullptr, 0, 0, sink, softcap, DV, gate_ch, st);
     return CM_ERR_DTYPE;
 }
 
@@ -476,7 +484,7 @@ extern "C" int cm_attn_append_simt(int dt, void* ctx, long long ldc, const void*
                                    const int* seq_start, const int* seq_pos0, const int* seq_slot, const void* pool,
                                    long long pages, const int* ptab, long long ptab_stride, int ring, int B,
                                    int max_len, int QH, int KVH, int HD, int window, float scale, float softcap,
-                                   const float* sink, cudaStream_t st) {
+                                   const float* sink, int DV, int gate_ch, cudaStream_t st) {
     if (B <= 0 || max_len <= 0) return CM_OK;
     if (HD > 32 * AP_MAXJ) CM_REFUSE("attn_append: head size %d above %d", HD, 32 * AP_MAXJ);
     if (QH % KVH) CM_REFUSE("attn_append: %d query heads over %d key heads", QH, KVH);
@@ -484,10 +492,10 @@ extern "C" int cm_attn_append_simt(int dt, void* ctx, long long ldc, const void*
     if (!seq_pos0 || !seq_slot || !pool || !ptab) CM_REFUSE("attn_append: positions, slots, cache and page table are needed");
     if (dt == DT_F32)
         return launch_attn_simt<float, true>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, QH, KVH, HD, window,
-                                             scale, seq_pos0, seq_slot, pool, pages, ptab, (int)ptab_stride, ring, sink, softcap, st);
+                                             scale, seq_pos0, seq_slot, pool, pages, ptab, (int)ptab_stride, ring, sink, softcap, DV, gate_ch, st);
     if (dt == DT_BF16)
         return launch_attn_simt<bf16, true>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, QH, KVH, HD, window,
-                                            scale, seq_pos0, seq_slot, pool, pages, ptab, (int)ptab_stride, ring, sink, softcap, st);
+                                            scale, seq_pos0, seq_slot, pool, pages, ptab, (int)ptab_stride, ring, sink, softcap, DV, gate_ch, st);
     return CM_ERR_DTYPE;
 }
 
@@ -757,14 +765,14 @@ attn_decode_kernel(float* __restrict__ part_o, float* __restrict__ part_ml, cons
     }
 }
 
-// Merge of the chunks of one (sequence, head), in chunk order; gate; store.
+// Merge of the chunks of one (sequence, head), in chunk order; gate; store (see the gate's two forms above).
 template <typename T>
 __global__ void attn_decode_merge_kernel(T* __restrict__ ctx, long long ldc,
                                          const float* __restrict__ part_o,
                                          const float* __restrict__ part_ml,
                                          const T* __restrict__ gate, long long ldg,
                                          const int* __restrict__ seq_pos, int ring, int QH, int HD,
-                                         int n_chunks, const float* __restrict__ sink) {
+                                         int n_chunks, const float* __restrict__ sink, int DV, int gate_ch) {
     pdl_trigger();
     pdl_wait();
     const int hq = blockIdx.x, b = blockIdx.y;
@@ -781,14 +789,15 @@ __global__ void attn_decode_merge_kernel(T* __restrict__ ctx, long long ldc,
     }
     if (sink) den += expf(sink[hq] - mx);          // the sink has no key and no value: it counts once, here
     float g = 1.f;
-    if (gate) g = sigmoid_f32(to_f32(gate[(long long)b * ldg + hq]));
-    for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+    if (gate && !gate_ch) g = sigmoid_f32(to_f32(gate[(long long)b * ldg + hq]));
+    for (int d = threadIdx.x; d < DV; d += blockDim.x) {
+        if (gate && gate_ch) g = sigmoid_f32(to_f32(gate[(long long)b * ldg + (long long)hq * DV + d]));
         float o = 0.f;
         for (int c = 0; c < nc; ++c) {
             const float mc = part_ml[(base + c) * 2];
             if (mc != -INFINITY) o += part_o[(base + c) * HD + d] * expf(mc - mx);
         }
-        ctx[(long long)b * ldc + (long long)hq * HD + d] = from_f32<T>(o / den * g);
+        ctx[(long long)b * ldc + (long long)hq * DV + d] = from_f32<T>(o / den * g);
     }
 }
 
@@ -808,13 +817,15 @@ extern "C" int cm_attn_decode(int dt, void* ctx, long long ldc, const void* q, l
                               const void* gate, long long ldg, const int* seq_pos, const int* seq_slot,
                               const void* pool, long long pages, const int* ptab, int ptab_stride,
                               int ring, int window, int B, int QH, int KVH, int HD, int n_chunks,
-                              float scale, float softcap, float* part_o, float* part_ml, const float* sink, cudaStream_t st) {
+                              float scale, float softcap, float* part_o, float* part_ml, const float* sink, int DV, int gate_ch,
+                              cudaStream_t st) {
     if (B <= 0) return CM_OK;
     if (HD % 8 || HD < 8 || HD > CM_MAX_HEAD_DIM)
         CM_REFUSE("attn_decode: head size %d (multiples of 8 up to %d)", HD, CM_MAX_HEAD_DIM);
     if (QH % KVH) CM_REFUSE("attn_decode: %d query heads over %d key heads", QH, KVH);
     if (ring % PAGE_TOKENS) CM_REFUSE("attn_decode: ring of %d entries is no multiple of %d", ring, PAGE_TOKENS);
     if (n_chunks <= 0) CM_REFUSE("attn_decode: %d chunks", n_chunks);
+    if (DV < 1 || DV > HD) CM_REFUSE("attn_decode: %d of %d channels stored", DV, HD);
     const int G = QH / KVH;
     const int gb = G >= 8 ? 8 : (G >= 4 ? 4 : (G >= 2 ? 2 : 1));
     const int groups = AD_THREADS / (HD / 8);
@@ -843,17 +854,17 @@ extern "C" int cm_attn_decode(int dt, void* ctx, long long ldc, const void* q, l
                                                 &n_parts, st);
         if (rc != CM_OK) return rc;
         cm_launch(attn_decode_merge_kernel<bf16>, mgrid, mthreads, 0, st, (bf16*)ctx, ldc, part_o, part_ml,
-                  (const bf16*)gate, ldg, seq_pos, ring, QH, HD, n_parts, sink);
+                  (const bf16*)gate, ldg, seq_pos, ring, QH, HD, n_parts, sink, DV, gate_ch);
     } else if (dt == DT_F32) {
         AD_DISPATCH(float);
         CM_CHECK_LAUNCH();
         cm_launch(attn_decode_merge_kernel<float>, mgrid, mthreads, 0, st, (float*)ctx, ldc, part_o, part_ml,
-                  (const float*)gate, ldg, seq_pos, ring, QH, HD, n_chunks, sink);
+                  (const float*)gate, ldg, seq_pos, ring, QH, HD, n_chunks, sink, DV, gate_ch);
     } else if (dt == DT_BF16) {
         AD_DISPATCH(bf16);
         CM_CHECK_LAUNCH();
         cm_launch(attn_decode_merge_kernel<bf16>, mgrid, mthreads, 0, st, (bf16*)ctx, ldc, part_o, part_ml,
-                  (const bf16*)gate, ldg, seq_pos, ring, QH, HD, n_chunks, sink);
+                  (const bf16*)gate, ldg, seq_pos, ring, QH, HD, n_chunks, sink, DV, gate_ch);
     } else
         return CM_ERR_DTYPE;
 #undef AD_DISPATCH
@@ -918,5 +929,5 @@ extern "C" int cm_attn_decode_noalloc(int dt, void* ctx, long long ldc, const vo
     if (rc != CM_OK) return rc;
     // part_o first (16-byte aligned for any size since HD is a multiple of 8), then part_ml
     return cm_attn_decode(dt, ctx, ldc, q, ldq, gate, ldg, seq_pos, seq_slot, pool, pages, ptab, ptab_stride, ring,
-                          window, B, QH, KVH, HD, n_chunks, scale, 0.f, scratch, scratch + o_floats, nullptr, st);
+                          window, B, QH, KVH, HD, n_chunks, scale, 0.f, scratch, scratch + o_floats, nullptr, HD, 0, st);
 }

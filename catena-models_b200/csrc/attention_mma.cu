@@ -64,7 +64,7 @@ attn_prefill_mma_kernel(bf16* __restrict__ ctx, long long ldc, const bf16* __res
                         int KVH, int window, float scale_log2, const int* __restrict__ seq_pos0,
                         const int* __restrict__ seq_slot, const bf16* __restrict__ pool, long long pages,
                         const int* __restrict__ ptab, int ptab_stride, int ring, const float* __restrict__ sink,
-                        float cap_in) {
+                        float cap_in, int DV, int gate_ch) {
     // cap_in > 0: the scores are bounded, s <- cap tanh(s scale / cap); cap_in = scale / cap, and scale_log2 is then cap log2 e
     constexpr int LDS = HD + 8;                   // padded row, elements
     constexpr int CH = HD / 8;                    // 16-byte chunks per row
@@ -292,11 +292,21 @@ attn_prefill_mma_kernel(bf16* __restrict__ ctx, long long ldc, const bf16* __res
         const long long tok = s0 + row - p0;
         // a sink logit (natural units; the running maximum is in log2 units) joins the denominator only
         float f = 1.f / (l_run[h] + (sink ? exp2f(sink[hq] * 1.4426950408889634f - m_run[h]) : 0.f));
-        if (gate) f *= sigmoid_f32(__bfloat162float(gate[tok * ldg + hq]));
-        bf16* dst = ctx + tok * ldc + (long long)hq * HD;
+        if (gate && !gate_ch) f *= sigmoid_f32(__bfloat162float(gate[tok * ldg + hq]));
+        bf16* dst = ctx + tok * ldc + (long long)hq * DV;
+        const bf16* gr = gate + tok * ldg + (long long)hq * DV;
 #pragma unroll
-        for (int j = 0; j < HD / 8; ++j)
-            *reinterpret_cast<uint32_t*>(dst + 8 * j + 2 * t) = pack_bf16(o[j][2 * h] * f, o[j][2 * h + 1] * f);
+        for (int j = 0; j < HD / 8; ++j) {
+            const int d = 8 * j + 2 * t;
+            if (d >= DV) continue;                             // DV is even
+            float lo = o[j][2 * h] * f, hi = o[j][2 * h + 1] * f;
+            if (gate && gate_ch) {
+                const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr + d));
+                lo *= sigmoid_f32(z.x);
+                hi *= sigmoid_f32(z.y);
+            }
+            *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16(lo, hi);
+        }
     }
 }
 
@@ -310,6 +320,8 @@ struct FaPast {                      // where the keys and values below a sequen
     int ring;
     const float* sink;               // per query head, or null: a logit without key and value in the softmax's denominator
     float softcap;                   // > 0: scores bounded to (-softcap, softcap) by a tanh
+    int DV;                          // channels of a head that are stored (even)
+    int gate_ch;                     // the gate has a logit per stored channel, not per head
 };
 
 template <int HD, int BQ, bool PAST>
@@ -331,7 +343,7 @@ static int launch_fa_bq(void* ctx, long long ldc, const void* q, const void* k, 
               (const bf16*)gate, ldg, seq_start, QH, KVH, window,
               (past.softcap > 0.f ? past.softcap : scale) * 1.4426950408889634f, past.seq_pos0,
               past.seq_slot, (const bf16*)past.pool, past.pages, past.ptab, past.ptab_stride, past.ring, past.sink,
-              past.softcap > 0.f ? scale / past.softcap : 0.f);
+              past.softcap > 0.f ? scale / past.softcap : 0.f, past.DV, past.gate_ch);
     CM_CHECK_LAUNCH();
     return CM_OK;
 }
@@ -359,6 +371,8 @@ static int dispatch_fa(void* ctx, long long ldc, const void* q, const void* k, c
     if (QH % KVH) CM_REFUSE("attn_prefill_mma: %d query heads over %d key heads", QH, KVH);
     if (ld % 8 || ldc % 2 || ((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)past.pool) & 15 || (uintptr_t)ctx & 3)
         CM_REFUSE("attn_prefill_mma: row pitch %lld must be a multiple of 8 and the operands 16-byte aligned", ld);
+    if (past.DV < 2 || past.DV > HD || past.DV % 2 || (past.gate_ch && (ldg % 2 || (uintptr_t)gate & 3)))
+        CM_REFUSE("attn_prefill_mma: %d of %d channels stored (an even number; gate rows aligned to 4 bytes)", past.DV, HD);
 #define FA_CASE(D) \
     case D: return launch_fa<D, PAST>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, QH, KVH, window, scale, past, st);
     switch (HD) {
@@ -373,9 +387,9 @@ static int dispatch_fa(void* ctx, long long ldc, const void* q, const void* k, c
 extern "C" int cm_attn_prefill_mma(void* ctx, long long ldc, const void* q, const void* k, const void* v,
                                    long long ld, const void* gate, long long ldg, const int* seq_start, int B,
                                    int max_len, int QH, int KVH, int HD, int window, float scale, float softcap,
-                                   const float* sink, cudaStream_t st) {
+                                   const float* sink, int DV, int gate_ch, cudaStream_t st) {
     if (B <= 0 || max_len <= 0) return CM_OK;
-    const FaPast none = {nullptr, nullptr, nullptr, 0, nullptr, 0, 0, sink, softcap};
+    const FaPast none = {nullptr, nullptr, nullptr, 0, nullptr, 0, 0, sink, softcap, DV, gate_ch};
     return dispatch_fa<false>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, QH, KVH, HD, window, scale, none, st);
 }
 
@@ -385,12 +399,13 @@ extern "C" int cm_attn_append_mma(void* ctx, long long ldc, const void* q, const
                                   long long ld, const void* gate, long long ldg, const int* seq_start,
                                   const int* seq_pos0, const int* seq_slot, const void* pool, long long pages,
                                   const int* ptab, long long ptab_stride, int ring, int B, int max_len, int QH, int KVH,
-                                  int HD, int window, float scale, float softcap, const float* sink, cudaStream_t st) {
+                                  int HD, int window, float scale, float softcap, const float* sink, int DV, int gate_ch,
+                                  cudaStream_t st) {
     if (B <= 0 || max_len <= 0) return CM_OK;
     if (ring % PAGE_TOKENS) CM_REFUSE("attn_append_mma: ring of %d entries is no multiple of %d", ring, PAGE_TOKENS);
     if (!seq_pos0 || !seq_slot || !pool || !ptab)
         CM_REFUSE("attn_append_mma: positions, slots, cache and page table are needed");
-    const FaPast past = {seq_pos0, seq_slot, pool, pages, ptab, (int)ptab_stride, ring, sink, softcap};
+    const FaPast past = {seq_pos0, seq_slot, pool, pages, ptab, (int)ptab_stride, ring, sink, softcap, DV, gate_ch};
     return dispatch_fa<true>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, QH, KVH, HD, window, scale, past, st);
 }
 

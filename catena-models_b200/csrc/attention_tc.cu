@@ -166,7 +166,23 @@ struct FtPast {                      // where the keys and values below a sequen
     const float* sink;               // per query head, or null: a logit without key and value in the softmax's denominator
     float softcap;                   // > 0: scores bounded to (-softcap, softcap) by a tanh, and
     float cap_in;                    // scale / softcap, what a raw score is multiplied by inside the tanh (0: no bound)
+    int DV;                          // channels of a head that are stored, side by side (a multiple of 8)
+    int gate_ch;                     // the gate has a logit per stored channel, not per head
 };
+
+// Eight finished channels of a row, times their gates when those come per channel (gr: the row's and head's logits).
+__device__ __forceinline__ void ft_store8(bf16* dst, const bf16* gr, bool gate_ch, const float* v) {
+    float out[8];
+    if (gate_ch) {
+        load8f<bf16>(gr, out);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) out[e] = __fdividef(v[e], 1.f + __expf(-out[e]));
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) out[e] = v[e];
+    }
+    store8f<bf16>(dst, out);
+}
 
 // One work item: a 128-query tile of one query head of one sequence, and the key tiles it takes.
 struct FtItem {
@@ -673,19 +689,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                 float f = 1.f / (l_run * f_mine + other.y * f_theirs +
                                  (past.sink ? exp2f(past.sink[it.hq] * 1.4426950408889634f - m) : 0.f));
                 const long long tok = it.s0 + row_l;
-                if (gate) f *= sigmoid_f32(__bfloat162float(gate[tok * ldg + it.hq]));
-                bf16* dst = ctx + tok * ldc + (long long)it.hq * HD + g * HALF;
+                const bool gate_ch = gate && past.gate_ch;
+                if (gate && !gate_ch) f *= sigmoid_f32(__bfloat162float(gate[tok * ldg + it.hq]));
+                const long long col = (long long)it.hq * past.DV + g * HALF;
+                bf16* dst = ctx + tok * ldc + col;
+                const bf16* gr = gate + tok * ldg + col;
 #pragma unroll
                 for (int c = 0; c < HALF / 8; ++c) {
-                    uint4 raw;
-                    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+                    if (g * HALF + 8 * c >= past.DV) continue;
+                    float v[8];
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        const int d = 8 * c + 2 * e;
-                        h[e] = __floats2bfloat162_rn((mine[d] * f_mine + theirs[d] * f_theirs) * f,
-                                                     (mine[d + 1] * f_mine + theirs[d + 1] * f_theirs) * f);
-                    }
-                    *reinterpret_cast<uint4*>(dst + 8 * c) = raw;
+                    for (int e = 0; e < 8; ++e) v[e] = (mine[8 * c + e] * f_mine + theirs[8 * c + e] * f_theirs) * f;
+                    ft_store8(dst + 8 * c, gr + 8 * c, gate_ch, v);
                 }
             }
             ++i;
@@ -763,6 +778,8 @@ static int launch_ft(void* ctx, long long ldc, const void* q, const void* k, con
     }
     int tiles_x = (max_len + FT_TILE - 1) / FT_TILE;
     if (const int ct = ft_chunk_tiles(window, tiles_x); ct > 1) tiles_x = (tiles_x + ct - 1) / ct * ct;      // whole chunks: see ft_item
+    if (past.DV < 8 || past.DV > HD || past.DV % 8 || (past.gate_ch && (ldg % 8 || (uintptr_t)gate & 15)))
+        CM_REFUSE("attn_prefill_tc: %d of %d channels stored (a multiple of 8; gate rows aligned to 16 bytes)", past.DV, HD);
     const long long items = (long long)tiles_x * QH * B;
     if (items > 0x7fffffffLL) CM_REFUSE("attn_prefill_tc: %lld items", items);
     const long long blocks = SOLO ? (items + 1) / 2 : items;
@@ -788,12 +805,12 @@ static int launch_ft(void* ctx, long long ldc, const void* q, const void* k, con
 extern "C" int cm_attn_prefill_tc(void* ctx, long long ldc, const void* q, const void* k, const void* v, long long ld,
                                   const void* gate, long long ldg, const int* seq_start, int B, int max_len,
                                   long long T, int QH, int KVH, int HD, int window, float scale, float softcap,
-                                  const float* sink, int* err, cudaStream_t st) {
+                                  const float* sink, int DV, int gate_ch, int* err, cudaStream_t st) {
     if (B <= 0 || max_len <= 0) return CM_OK;
     if (QH % KVH) CM_REFUSE("attn_prefill_tc: %d query heads over %d key heads", QH, KVH);
     if (ld % 8 || ldc % 8 || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)ctx) & 15))
         CM_REFUSE("attn_prefill_tc: row pitches %lld, %lld must be multiples of 8 and the operands 16-byte aligned", ld, ldc);
-    const FtPast none = {nullptr, nullptr, nullptr, 0, 0, 0, sink, softcap, softcap > 0.f ? scale / softcap : 0.f};
+    const FtPast none = {nullptr, nullptr, nullptr, 0, 0, 0, sink, softcap, softcap > 0.f ? scale / softcap : 0.f, DV, gate_ch};
     if (HD == 64)
         return launch_ft<64, FT_STAGES_64, false>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, T, QH, KVH, window, scale,
                                        none, nullptr, err, st);
@@ -811,7 +828,8 @@ extern "C" int cm_attn_append_tc(void* ctx, long long ldc, const void* q, const 
                                  const void* gate, long long ldg, const int* seq_start, const int* seq_pos0,
                                  const int* seq_slot, const void* pool, long long pages, const int* ptab,
                                  long long ptab_stride, int ring, int B, int max_len, long long T, int QH, int KVH,
-                                 int HD, int window, float scale, float softcap, const float* sink, int* err, cudaStream_t st) {
+                                 int HD, int window, float scale, float softcap, const float* sink, int DV, int gate_ch, int* err,
+                                 cudaStream_t st) {
     if (B <= 0 || max_len <= 0) return CM_OK;
     if (QH % KVH) CM_REFUSE("attn_append_tc: %d query heads over %d key heads", QH, KVH);
     if (ring % PAGE_TOKENS) CM_REFUSE("attn_append_tc: ring of %d entries is no multiple of %d", ring, PAGE_TOKENS);
@@ -820,7 +838,7 @@ extern "C" int cm_attn_append_tc(void* ctx, long long ldc, const void* q, const 
     if (ld % 8 || ldc % 8 || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)ctx | (uintptr_t)pool) & 15))
         CM_REFUSE("attn_append_tc: row pitches %lld, %lld must be multiples of 8 and the operands 16-byte aligned", ld, ldc);
     if (2 * pages * KVH * PAGE_TOKENS > 0x7fffffffLL) CM_REFUSE("attn_append_tc: a cache of %lld pages is too large", pages);
-    const FtPast past = {seq_pos0, seq_slot, ptab, ptab_stride, pages, ring, sink, softcap, softcap > 0.f ? scale / softcap : 0.f};
+    const FtPast past = {seq_pos0, seq_slot, ptab, ptab_stride, pages, ring, sink, softcap, softcap > 0.f ? scale / softcap : 0.f, DV, gate_ch};
     if (HD == 64)
         return launch_ft<64, FT_STAGES_64, true>(ctx, ldc, q, k, v, ld, gate, ldg, seq_start, B, max_len, T, QH, KVH, window, scale,
                                       past, pool, err, st);

@@ -396,15 +396,17 @@ attn_prefill_tc_solo_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 // a sink logit (natural units; m_ref is in log2 units) joins the denominator only
                 float f = 1.f / (l_run + (past.sink ? exp2f(past.sink[it.hq] * 1.4426950408889634f - m_ref) : 0.f));
                 const long long tok = it.s0 + row_l;
-                if (gate) f *= sigmoid_f32(__bfloat162float(gate[tok * ldg + it.hq]));
-                bf16* dst = ctx + tok * ldc + (long long)it.hq * HD;
+                const bool gate_ch = gate && past.gate_ch;
+                if (gate && !gate_ch) f *= sigmoid_f32(__bfloat162float(gate[tok * ldg + it.hq]));
+                bf16* dst = ctx + tok * ldc + (long long)it.hq * past.DV;
+                const bf16* gr = gate + tok * ldg + (long long)it.hq * past.DV;
 #pragma unroll
                 for (int c = 0; c < HD / 8; ++c) {
-                    uint4 raw;
-                    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+                    if (8 * c >= past.DV) continue;
+                    float v[8];
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) h[e] = __floats2bfloat162_rn(o[8 * c + 2 * e] * f, o[8 * c + 2 * e + 1] * f);
-                    *reinterpret_cast<uint4*>(dst + 8 * c) = raw;
+                    for (int e = 0; e < 8; ++e) v[e] = o[8 * c + e] * f;
+                    ft_store8(dst + 8 * c, gr + 8 * c, gate_ch, v);
                 }
             }
         }

@@ -198,6 +198,15 @@ __device__ __forceinline__ float gated_act(float g, float u, int act, float limi
     return g * sigmoid_f32(g) * u;
 }
 
+// The tanh form of gelu as a plain activation: 0.5 z (1 + tanh(u)) = z / (1 + e^(-2u)), u = sqrt(2/pi) (z + 0.044715 z^3).
+__device__ __forceinline__ float gelu_tanh_f32(float z) {
+    return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+// The same from one exponential and one division, for epilogues that round the result to bfloat16.
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+    return __fdividef(z, 1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+
 // Eight consecutive elements as floats: one 16-byte access for bfloat16, two for float.
 template <typename T>
 __device__ __forceinline__ void load8f(const T* p, float* out);

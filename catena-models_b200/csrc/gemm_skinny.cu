@@ -24,6 +24,7 @@ namespace cg = cooperative_groups;
 #define SK_MODE_GEGLU 3                      // as SWIGLU with the tanh form of gelu on the gate
 #define SK_MODE_CLAMPED 4                    // both halves clamped at a limit L: min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1)
 #define SK_GATED(M) ((M) == SK_MODE_SWIGLU || (M) == SK_MODE_GEGLU || (M) == SK_MODE_CLAMPED)
+#define SK_MODE_GELU 5                       // no gate: the tanh form of gelu on every output
 #define SK_MODE_PARTS 2          // float partial sums per k-slice, no exchange between the blocks of a row tile
 
 __device__ __forceinline__ void mma_bf16_16816(float* d, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
@@ -188,7 +189,7 @@ gemm_skinny_kernel(TY* __restrict__ Y, const bf16* __restrict__ X, const bf16* _
                 const float ag = MODE == SK_MODE_GEGLU ? 0.5f * gr * (1.f + th) : gr * sigmoid_f32(gr);
                 Y[(long long)m * ldy + row] = from_f32<TY>(ag * ur);
             } else {
-                Y[(long long)m * ldy + row] = from_f32<TY>(tot[0]);
+                Y[(long long)m * ldy + row] = from_f32<TY>(MODE == SK_MODE_GELU ? gelu_tanh_fast(tot[0]) : tot[0]);
             }
         }
     }
@@ -378,6 +379,10 @@ extern "C" int cm_gemm_skinny(int dty, void* Y, const void* X, const void* W, in
         CM_REFUSE("gemm_skinny: inner size %d and row strides %lld, %lld must be multiples of 8", K, ldx, ldw);
     if ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W)) & 15)
         CM_REFUSE("gemm_skinny: operands must be 16-byte aligned");
+    if (swiglu == 4) {                       // no gate: W has N rows
+        if (dty != DT_BF16) return CM_ERR_DTYPE;
+        return dispatch_skinny<bf16, SK_MODE_GELU>(Y, X, W, M, N, K, ldx, ldw, ldy, st);
+    }
     if (swiglu) {
         if (dty != DT_BF16) return CM_ERR_DTYPE;
         if (swiglu == 2) return dispatch_skinny<bf16, SK_MODE_GEGLU>(Y, X, W, M, N, K, ldx, ldw, ldy, st);

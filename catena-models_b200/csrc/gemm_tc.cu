@@ -36,7 +36,8 @@ static_assert(TC_BM == CM_FEW_ROWS_MAX_ROWS, "cm_limits.h: CM_FEW_ROWS_MAX_ROWS"
 #define TC_MODE_SWIGLU 1
 #define TC_MODE_GEGLU 2                      // as SWIGLU with the tanh form of gelu on the gate
 #define TC_MODE_CLAMPED 3                    // both halves clamped at a limit L: min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1)
-#define TC_GATED(M) ((M) != TC_MODE_PLAIN)
+#define TC_MODE_GELU 4                       // no gate: the tanh form of gelu on every output
+#define TC_GATED(M) ((M) != TC_MODE_PLAIN && (M) != TC_MODE_GELU)
 
 // What the gate passes through before it meets the up half.
 template <int MODE>
@@ -274,6 +275,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                                 const float g = rounded<TC>(v[i]), uu = rounded<TC>(u[i]);
                                 v[i] = tc_gated<MODE>(g, uu, gate_limit);
                             }
+                        } else if (MODE == TC_MODE_GELU) {
+#pragma unroll
+                            for (int i = 0; i < 32; ++i) v[i] = gelu_tanh_fast(v[i]);
                         }
                         if (tma_store) {
                             stage_cols(sbuf, r_tile, h * (32 * (int)sizeof(TC) / 16), v, (TC*)nullptr);
@@ -549,6 +553,9 @@ gemm_tc_splitk_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
                     o[i] = tc_gated<MODE>(g, u, gate_limit);
                 }
                 if (lane >= 16) continue;
+            } else if (MODE == TC_MODE_GELU) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) o[i] = gelu_tanh_fast(o[i]);
             }
             TC* dst = C + (long long)row * ldc + col;
             if (vec_ok && col + 3 < N) {
@@ -752,7 +759,8 @@ static int launch_splitk_rows(void* C, const void* A, const void* B, int M, int 
 }
 
 // A [M,K] and B [N,K] (2N rows when swiglu) bfloat16, row pitches lda/ldb multiples of 8
-// elements, bases 16-byte aligned; C bfloat16 or float.  block_n: 256 (128 x 256 tiles, four
+// elements, bases 16-byte aligned; C bfloat16 or float.  swiglu: 0 none, 1 silu(g) u, 2 the tanh form of gelu on g, 3 the
+// clamped gate, 4 no gate but the tanh form of gelu on every output (B has N rows).  block_n: 256 (128 x 256 tiles, four
 // stages: the most arithmetic per byte moved), 128 (128 x 128 tiles, six stages: twice as
 // many tiles, for products with few rows where the number of tiles decides how many SMs stream
 // weights) or 192 (plain bfloat16 products whose tiles then fill their rounds over the SMs better).  err: device int, raised by a block whose pipeline wait ran out; may be null.
@@ -764,6 +772,12 @@ extern "C" int cm_gemm_tc(int dtc, void* C, const void* A, const void* B, int M,
     if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B)) & 15)
         CM_REFUSE("gemm_tc: operands must be 16-byte aligned");
     if (block_n != 128 && block_n != 192 && block_n != 256) CM_REFUSE("gemm_tc: tile width %d (128, 192 or 256)", block_n);
+    if (swiglu == 4) {
+        if (dtc != DT_BF16) return CM_ERR_DTYPE;
+        if (block_n == 256) return launch_tc<256, 4, bf16, TC_MODE_GELU>(C, A, B, M, N, K, lda, ldb, ldc, err, st);
+        if (block_n == 192) return launch_tc<192, 4, bf16, TC_MODE_GELU>(C, A, B, M, N, K, lda, ldb, ldc, err, st);
+        return launch_tc<128, 6, bf16, TC_MODE_GELU>(C, A, B, M, N, K, lda, ldb, ldc, err, st);
+    }
     if (block_n == 192 && (swiglu || dtc != DT_BF16)) CM_REFUSE("gemm_tc: 192-wide tiles are for plain bfloat16 products");
     if (swiglu) {
         if (dtc != DT_BF16) return CM_ERR_DTYPE;
@@ -802,7 +816,7 @@ extern "C" int cm_gemm_tc_grouped(int dtc, void* C, const void* A, const void* B
         CM_REFUSE("gemm_tc_grouped: operands must be 16-byte aligned");
     if (!tile_group || groups < 1) CM_REFUSE("gemm_tc_grouped: the row tiles' groups are missing");
     if (block_n != 128 && block_n != 256) CM_REFUSE("gemm_tc_grouped: tile width %d (128 or 256)", block_n);
-    if (swiglu == 2) CM_REFUSE("gemm_tc_grouped: the gated form has silu and the clamped gate only");
+    if (swiglu == 2 || swiglu == 4) CM_REFUSE("gemm_tc_grouped: the gated form has silu and the clamped gate only");
     if (swiglu == 3) {
         if (dtc != DT_BF16) return CM_ERR_DTYPE;
         if (!(gate_limit > 0.f)) CM_REFUSE("gemm_tc_grouped: the clamped gate needs a positive limit");
@@ -887,7 +901,10 @@ extern "C" int cm_gemm_tc_few_rows(int dtc, void* C, const void* A, const void* 
     if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(B)) & 15)
         CM_REFUSE("gemm_tc: operands must be 16-byte aligned");
     int rc;
-    if (swiglu) {
+    if (swiglu == 4) {
+        if (dtc != DT_BF16) return CM_ERR_DTYPE;
+        rc = launch_splitk<bf16, TC_MODE_GELU>(C, A, B, M, N, K, lda, ldb, ldc, splits, err, st);
+    } else if (swiglu) {
         if (dtc != DT_BF16) return CM_ERR_DTYPE;
         if (swiglu == 3 && !(gate_limit > 0.f)) CM_REFUSE("gemm_tc_few_rows: the clamped gate needs a positive limit");
         rc = swiglu == 3 ? launch_splitk<bf16, TC_MODE_CLAMPED>(C, A, B, M, N, K, lda, ldb, ldc, splits, err, st, nullptr, 0, gate_limit)
@@ -908,7 +925,7 @@ extern "C" int cm_gemm_tc_few_rows(int dtc, void* C, const void* A, const void* 
     int sm_count = 0, dev = 0;
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev);
-    const int out_cols = swiglu ? 64 : 128;
+    const int out_cols = swiglu && swiglu != 4 ? 64 : 128;
     const int tiles = (N + out_cols - 1) / out_cols;
     const int width = (dtc == DT_BF16 && sm_count > 0 && tiles > sm_count && tiles <= 2 * sm_count) ? 256 : 128;
     return cm_gemm_tc(dtc, C, A, B, M, N, K, lda, ldb, ldc, swiglu, width, err, gate_limit, st);

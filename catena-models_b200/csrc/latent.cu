@@ -12,8 +12,10 @@
 // same cache entries, and the weighted sum runs over the latents.  The two per-head products (W_uk^T on the queries,
 // W_uv on the sums) are `head_linear`.  Norms, angles, scores, softmax and the sums over them are float.
 //
-// Every kind of step writes its entries first and then reads all keys from the cache: whole prompts, portions,
-// single tokens and mixed batches are one code path.  Rows of padding (tok_seq < 0) are left alone.
+// Without a window every kind of step writes its entries first and then reads all keys from the cache: whole prompts,
+// portions, single tokens and mixed batches are one code path.  With a window the cache is a ring, and a step of more than
+// one token a sequence reads its own positions from the entries kept side by side (`ckv`) and older ones from the ring.
+// Rows of padding (tok_seq < 0) are left alone.
 #include "common.cuh"
 #include "latent.h"
 #include <math.h>
@@ -35,8 +37,8 @@ latent_prepare_kernel(const LatentArgs a) {
         return;
     }
     const T* row = (const T*)a.proj + t * a.ld_proj;
-    // the query latent
-    {
+    // the query latent (a layer whose queries come straight from the input has none)
+    if (a.QR > 0) {
         const T* x = row + a.q_off;
         float ss = 0.f;
         for (int c = threadIdx.x; c < a.QR; c += blockDim.x) {
@@ -51,8 +53,16 @@ latent_prepare_kernel(const LatentArgs a) {
     if (a.no_entry) return;
     // the cache entry
     const int pos = a.tok_pos[t];
-    const int page = a.ptab[(long long)a.seq_slot[b] * a.ptab_stride + pos / PAGE_TOKENS];
-    T* entry = (T*)a.pool + ((long long)page * PAGE_TOKENS + pos % PAGE_TOKENS) * a.EC;
+    T* entry = nullptr;                               // a ring keeps the last `ring` positions of a sequence
+    if (!a.no_store && (a.ring == 0 || pos + a.ring >= a.seq_end[b])) {
+        const int e = a.ring ? pos % a.ring : pos;
+        const int page = a.ptab[(long long)a.seq_slot[b] * a.ptab_stride + e / PAGE_TOKENS];
+        entry = (T*)a.pool + ((long long)page * PAGE_TOKENS + e % PAGE_TOKENS) * a.EC;
+    }
+    auto put = [&](int c, T v) {                      // into the cache and beside the step's other entries
+        if (entry) entry[c] = v;
+        if (copy) copy[c] = v;
+    };
     const T* x = row + a.kv_off;
     float ss = 0.f;
     for (int c = threadIdx.x; c < a.KR; c += blockDim.x) {
@@ -61,11 +71,11 @@ latent_prepare_kernel(const LatentArgs a) {
     }
     ss = block_sum(ss, scratch);
     const float inv = 1.f / sqrtf(ss / (float)a.KR + a.eps);
-    for (int c = threadIdx.x; c < a.KR; c += blockDim.x) entry[c] = from_f32<T>((to_f32(x[c]) * inv) * a.wkv_norm[c]);
+    for (int c = threadIdx.x; c < a.KR; c += blockDim.x) put(c, from_f32<T>((to_f32(x[c]) * inv) * a.wkv_norm[c]));
     const T* r = x + a.KR;
     for (int i = threadIdx.x; i < (a.R + 1) / 2; i += blockDim.x) {
         if (2 * i + 1 >= a.R) {                       // an odd last channel has no partner
-            entry[a.KR + 2 * i] = r[2 * i];
+            put(a.KR + 2 * i, r[2 * i]);
             continue;
         }
         float sn, cs;
@@ -73,14 +83,40 @@ latent_prepare_kernel(const LatentArgs a) {
         sn *= a.mag;
         cs *= a.mag;
         const float u = to_f32(r[2 * i]), v = to_f32(r[2 * i + 1]);
-        entry[a.KR + 2 * i] = from_f32<T>(u * cs - v * sn);
-        entry[a.KR + 2 * i + 1] = from_f32<T>(v * cs + u * sn);
+        put(a.KR + 2 * i, from_f32<T>(u * cs - v * sn));
+        put(a.KR + 2 * i + 1, from_f32<T>(v * cs + u * sn));
     }
-    for (int c = a.KR + a.R + threadIdx.x; c < a.EC; c += blockDim.x) entry[c] = from_f32<T>(0.f);
-    if (copy) {
-        __syncthreads();                               // the entry is complete (every thread reads what others wrote)
-        for (int c = threadIdx.x; c < a.EC; c += blockDim.x) copy[c] = entry[c];
-    }
+    for (int c = a.KR + a.R + threadIdx.x; c < a.EC; c += blockDim.x) put(c, from_f32<T>(0.f));
+}
+
+// The step's entries, kept side by side so far, into the cache: the last part of a step that had to read the entries which
+// these rows replace.  One block per row.
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_store_kernel(const LatentArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const long long t = blockIdx.x;
+    const int b = a.tok_seq[t];
+    if (b < 0) return;
+    const int pos = a.tok_pos[t];
+    if (a.ring && pos + a.ring < a.seq_end[b]) return;
+    const int e = a.ring ? pos % a.ring : pos;
+    const int page = a.ptab[(long long)a.seq_slot[b] * a.ptab_stride + e / PAGE_TOKENS];
+    T* entry = (T*)a.pool + ((long long)page * PAGE_TOKENS + e % PAGE_TOKENS) * a.EC;
+    const T* src = (const T*)a.ckv + t * a.EC;
+    for (int c = threadIdx.x; c < a.EC; c += blockDim.x) entry[c] = src[c];
+}
+
+extern "C" int cm_latent_store(int dt, const LatentArgs* args, cudaStream_t st) {
+    const LatentArgs& a = *args;
+    if (a.rows <= 0) return CM_OK;
+    if (!a.ckv || a.ring % PAGE_TOKENS) CM_REFUSE("latent_store: the step's entries, and a ring of whole pages");
+    if (dt == DT_F32) cm_launch(latent_store_kernel<float>, (unsigned)a.rows, 128, 0, st, a);
+    else if (dt == DT_BF16) cm_launch(latent_store_kernel<bf16>, (unsigned)a.rows, 128, 0, st, a);
+    else return CM_ERR_DTYPE;
+    CM_CHECK_LAUNCH();
+    return CM_OK;
 }
 
 // The prompt form's operands: per row, queries, keys and values of every head in heads of HD channels, as the attention
@@ -206,6 +242,7 @@ __global__ void latent_query_turn_kernel(const LatentArgs a) {
 extern "C" int cm_latent_prepare(int dt, const LatentArgs* args, cudaStream_t st) {
     const LatentArgs& a = *args;
     if (a.rows <= 0) return CM_OK;
+    if (a.ring % PAGE_TOKENS || (a.no_store && !a.ckv)) CM_REFUSE("latent_prepare: a ring of %d entries, or no place for the entries", a.ring);
     if (a.EC < a.KR + a.R || a.EC % 8) CM_REFUSE("latent_prepare: entries of %d for %d + %d channels (a multiple of 8)", a.EC, a.KR, a.R);
     if (dt == DT_F32) cm_launch(latent_prepare_kernel<float>, (unsigned)a.rows, 128, 0, st, a);
     else if (dt == DT_BF16) cm_launch(latent_prepare_kernel<bf16>, (unsigned)a.rows, 128, 0, st, a);
@@ -235,7 +272,7 @@ extern "C" int cm_latent_query_turn(int dt, const LatentArgs* args, cudaStream_t
 template <typename TX, typename T, typename TY>
 __global__ void __launch_bounds__(256)
 head_linear_kernel(TY* __restrict__ y, const TX* __restrict__ x, const T* __restrict__ w, long long rows, int N, int K,
-                   long long ldx, long long ldy, int xs, int ys) {
+                   long long ldx, long long ldy, int xs, int ys, const T* __restrict__ gate, long long ldg) {
     __shared__ float sx[HL_BK][HL_TM + 4];
     __shared__ float sw[HL_BK][HL_TN + 4];
     pdl_trigger();
@@ -282,7 +319,9 @@ head_linear_kernel(TY* __restrict__ y, const TX* __restrict__ x, const T* __rest
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tc * 4 + j;
-            if (n < N) y[r * ldy + (long long)h * ys + n] = from_f32<TY>(acc[i][j]);
+            if (n >= N) continue;
+            const float g = gate ? sigmoid_f32(to_f32(gate[r * ldg + (long long)h * N + n])) : 1.f;
+            y[r * ldy + (long long)h * ys + n] = from_f32<TY>(acc[i][j] * g);
         }
     }
 }
@@ -293,7 +332,7 @@ head_linear_kernel(TY* __restrict__ y, const TX* __restrict__ x, const T* __rest
 template <typename TX, typename T, typename TY>
 __global__ void __launch_bounds__(256)
 head_linear_few_kernel(TY* __restrict__ y, const TX* __restrict__ x, const T* __restrict__ w, long long rows, int N, int K,
-                       long long ldx, long long ldy, int xs, int ys) {
+                       long long ldx, long long ldy, int xs, int ys, const T* __restrict__ gate, long long ldg) {
     pdl_trigger();
     pdl_wait();
     const int h = blockIdx.y, lane = threadIdx.x & 31;
@@ -314,22 +353,27 @@ head_linear_few_kernel(TY* __restrict__ y, const TX* __restrict__ x, const T* __
 #pragma unroll
         for (int r = 0; r < HL_FEW; ++r) {
             const float v = warp_sum(acc[r]);
-            if (lane == 0 && r0 + r < rows) y[(r0 + r) * ldy + (long long)h * ys + n] = from_f32<TY>(v);
+            if (lane == 0 && r0 + r < rows) {
+                const float g = gate ? sigmoid_f32(to_f32(gate[(r0 + r) * ldg + (long long)h * N + n])) : 1.f;
+                y[(r0 + r) * ldy + (long long)h * ys + n] = from_f32<TY>(v * g);
+            }
         }
     }
 }
 
+// gate (or null): a logit per row, head and column, gate[r][h * N + n] in the matrices' dtype; the result is multiplied by
+// its sigmoid.
 // x_f32 / y_f32: the rows read / written are float whatever the matrices' dtype (sums that stay unrounded between two steps).
 extern "C" int cm_head_linear(int dt, void* y, const void* x, const void* w, long long rows, int H, int N, int K, long long ldx,
-                              long long ldy, int xs, int ys, int x_f32, int y_f32, cudaStream_t st) {
+                              long long ldy, int xs, int ys, int x_f32, int y_f32, const void* gate, long long ldg, cudaStream_t st) {
     if (rows <= 0 || H <= 0 || N <= 0) return CM_OK;
     if (H > 65535) CM_REFUSE("head_linear: %d heads", H);
     const bool few = rows <= 2 * HL_FEW;
     dim3 grid(few ? (N + 7) / 8 : (N + HL_TN - 1) / HL_TN, few ? H : (unsigned)((rows + HL_TM - 1) / HL_TM), few ? 1 : H);
 #define HL_LAUNCH(TX, TW, TY) \
     do {                                                                                                                    \
-        if (few) cm_launch(head_linear_few_kernel<TX, TW, TY>, grid, 256, 0, st, (TY*)y, (const TX*)x, (const TW*)w, rows, N, K, ldx, ldy, xs, ys); \
-        else cm_launch(head_linear_kernel<TX, TW, TY>, grid, 256, 0, st, (TY*)y, (const TX*)x, (const TW*)w, rows, N, K, ldx, ldy, xs, ys);         \
+        if (few) cm_launch(head_linear_few_kernel<TX, TW, TY>, grid, 256, 0, st, (TY*)y, (const TX*)x, (const TW*)w, rows, N, K, ldx, ldy, xs, ys, (const TW*)gate, ldg); \
+        else cm_launch(head_linear_kernel<TX, TW, TY>, grid, 256, 0, st, (TY*)y, (const TX*)x, (const TW*)w, rows, N, K, ldx, ldy, xs, ys, (const TW*)gate, ldg);         \
     } while (0)
     if (dt == DT_F32) HL_LAUNCH(float, float, float);
     else if (dt == DT_BF16 && x_f32 && y_f32) HL_LAUNCH(float, bf16, float);
@@ -385,7 +429,9 @@ latent_attn_kernel(const LatentArgs a) {
     }
     const bool warp_live = r0 + warp * 4 < n_rows;    // a warp without rows (fewer heads than the block has rows) only fetches
     const int last_row = min(n_rows, r0 + LA_ROWS) - 1;
-    const int k_first = a.splits > 1 ? split * a.chunk : 0;
+    // the first key that any row of the block sees; key tiles begin at a multiple of LA_KT
+    const int first = first_visible(pos0 + r0 / H, a.window);
+    const int k_first = first / LA_KT * LA_KT + (a.splits > 1 ? split * a.chunk : 0);
     const int k_last = min(pos0 + last_row / H, a.splits > 1 ? k_first + a.chunk - 1 : 0x7fffffff);     // inclusive
     float mx[4], sum[4], acc[4][KRL];
 #pragma unroll
@@ -404,14 +450,14 @@ latent_attn_kernel(const LatentArgs a) {
             for (int e = threadIdx.x; e < LA_KT * E8; e += LA_THREADS) {
                 const int j = e / E8, c = (e - j * E8) * 8, kp = k0 + j;
                 float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-                if (kp < end) load8f<T>((const T*)a.pool + ((long long)ptab[kp / PAGE_TOKENS] * PAGE_TOKENS + kp % PAGE_TOKENS) * a.EC + c, v);
+                if (kp < end && kp >= first) load8f<T>(latent_entry<T>(a, ptab, s0, pos0, kp) + c, v);
 #pragma unroll
                 for (int x = 0; x < 8; ++x) sk[j * EK + c + x] = v[x];
             }
         } else {
             for (int e = threadIdx.x; e < LA_KT * E; e += LA_THREADS) {
                 const int j = e / E, c = e - j * E, kp = k0 + j;
-                sk[j * EK + c] = kp < end ? to_f32(((const T*)a.pool)[((long long)ptab[kp / PAGE_TOKENS] * PAGE_TOKENS + kp % PAGE_TOKENS) * a.EC + c]) : 0.f;
+                sk[j * EK + c] = kp < end && kp >= first ? to_f32(latent_entry<T>(a, ptab, s0, pos0, kp)[c]) : 0.f;
             }
         }
         __syncthreads();
@@ -435,7 +481,7 @@ latent_attn_kernel(const LatentArgs a) {
         float p[4];
 #pragma unroll
         for (int m = 0; m < 4; ++m) {
-            const bool seen = kp <= row_pos[m] && kp <= k_last;
+            const bool seen = kp <= row_pos[m] && kp <= k_last && kp >= first_visible(row_pos[m], a.window);
             const float sc = seen ? s[m] : -INFINITY;
             const float m_new = fmaxf(mx[m], warp_max(sc));
             const float ref = m_new == -INFINITY ? 0.f : m_new;
@@ -481,7 +527,7 @@ latent_attn_kernel(const LatentArgs a) {
             }
         } else {
             const float g = a.gate ? sigmoid_f32(to_f32(((const T*)a.gate)[t * a.ld_gate + h])) : 1.f;
-            const float f = g / sum[m];
+            const float f = g / (sum[m] + (a.sink ? expf(a.sink[h] - mx[m]) : 0.f));     // a sink joins the denominator only
             float* o = a.out + t * a.ldo + (long long)h * KR;
 #pragma unroll
             for (int ci = 0; ci < KRL; ++ci) {
@@ -528,6 +574,7 @@ latent_attn_merge_kernel(const LatentArgs a) {
     float sum = 0.f;
     for (int s = 0; s < a.splits; ++s) sum = fmaf(part[s * stride + 1], ws[s], sum);
     const float g = a.gate ? sigmoid_f32(to_f32(((const T*)a.gate)[t * a.ld_gate + h])) : 1.f;
+    if (a.sink) sum += expf(a.sink[h] - mx);          // the sink has no key and no value: it counts once, here
     const float f = g / sum;
     float* o = a.out + t * a.ldo + (long long)h * KR;
     for (int c = tid; c < KR; c += LA_MERGE_THREADS) {

@@ -2,6 +2,7 @@
 // record (kernels._LatentArgs).
 #pragma once
 #include <cuda_runtime.h>
+#include "cm_limits.h"
 
 struct LatentArgs {
     // the step's rows
@@ -40,7 +41,23 @@ struct LatentArgs {
     int HD, DV;
     float mag;                   // the factor on every sine and cosine (1: a plain rotation)
     int no_entry;                // latent_prepare: the layer reads another layer's entries; only the query latent is made
+    // a sliding window and a sink
+    int window;                  // > 0: a row sees the last `window` positions (itself among them); 0: every earlier one
+    int ring;                    // > 0: the cache keeps the last `ring` positions of a sequence, position p in entry p % ring
+    int no_store;                // latent_prepare: entries go to `ckv` only (a step that must first read what they replace)
+    const float* sink;           // [H] or null: a logit per head in the softmax's denominator, without key and value
 };
+
+#ifdef __CUDACC__
+// Where the entry of position kp lies, as the attention kernels read it: with `ckv` (the step's entries side by side) the
+// positions of the step come from there (row s0 + kp - pos0) and only older ones from the cache; a ring is indexed by kp % ring.
+template <typename T>
+__device__ __forceinline__ const T* latent_entry(const LatentArgs& a, const int* ptab, int s0, int pos0, int kp) {
+    if (a.ckv && kp >= pos0) return (const T*)a.ckv + (long long)(s0 + kp - pos0) * a.EC;
+    const int e = a.ring ? kp % a.ring : kp;
+    return (const T*)a.pool + ((long long)ptab[e / CM_PAGE_TOKENS] * CM_PAGE_TOKENS + e % CM_PAGE_TOKENS) * a.EC;
+}
+#endif
 
 // The splits' (maximum, sum, sums over the latents) of every (row, head) merged, normalised and gated (latent.cu); both
 // forms of the attention end with it.

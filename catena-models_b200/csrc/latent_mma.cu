@@ -87,7 +87,8 @@ latent_attn_mma_kernel(const LatentArgs a) {
         const int j = e / (LDK - EC), c = EC + e - j * (LDK - EC);
         Ks[j * LDK + c] = __float2bfloat16_rn(0.f);
     }
-    const int k_first = a.splits > 1 ? split * a.chunk : 0;
+    const int first = first_visible(pos, a.window);       // the first key that the row sees
+    const int k_first = first / LM_KT * LM_KT + (a.splits > 1 ? split * a.chunk : 0);
     const int k_last = min(pos, a.splits > 1 ? k_first + a.chunk - 1 : 0x7fffffff);        // inclusive
     const float scale_log2 = a.scale * 1.4426950408889634f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
@@ -105,17 +106,19 @@ latent_attn_mma_kernel(const LatentArgs a) {
     static_assert(PAGE_TOKENS % LM_KT == 0 && LM_THREADS == 4 * LM_KT, "a tile within a page, four threads an entry");
     auto fetch = [&](int k0, int buf, int page) {
         const int j = tid >> 2, kp = k0 + j;
-        const bool valid = kp < end && kp <= k_last;
-        const bf16* src = (const bf16*)a.pool + (valid ? ((long long)page * PAGE_TOKENS + kp % PAGE_TOKENS) * EC : 0);
+        const bool valid = kp < end && kp <= k_last && kp >= first;
+        const int row = (a.ring ? kp % a.ring : kp) % PAGE_TOKENS;
+        const bf16* src = (const bf16*)a.pool + (valid ? ((long long)page * PAGE_TOKENS + row) * EC : 0);
         bf16* dst = Ks + (buf * LM_KT + j) * LDK;
         for (int c8 = tid & 3; c8 < C8; c8 += 4) lm_copy16(dst + c8 * 8, src + (valid ? c8 * 8 : 0), valid);
         lm_copy_commit();
     };
+    auto page_of = [&](int k0) { return ptab[(a.ring ? k0 % a.ring : k0) / PAGE_TOKENS]; };      // a ring is whole pages: a tile lies within one
     const bool any = k_first <= k_last;
     int page_next = 0;
     if (any) {
-        fetch(k_first, 0, ptab[k_first / PAGE_TOKENS]);
-        if (k_first + LM_KT <= k_last) page_next = ptab[(k_first + LM_KT) / PAGE_TOKENS];
+        fetch(k_first, 0, page_of(k_first));
+        if (k_first + LM_KT <= k_last) page_next = page_of(k_first + LM_KT);
     }
     int buf = 0;
     for (int k0 = k_first; k0 <= k_last; k0 += LM_KT, buf ^= 1) {
@@ -123,7 +126,7 @@ latent_attn_mma_kernel(const LatentArgs a) {
         const bool more = k0 + LM_KT <= k_last;
         if (more) {
             fetch(k0 + LM_KT, buf ^ 1, page_next);
-            if (k0 + 2 * LM_KT <= k_last) page_next = ptab[(k0 + 2 * LM_KT) / PAGE_TOKENS];
+            if (k0 + 2 * LM_KT <= k_last) page_next = page_of(k0 + 2 * LM_KT);
         }
         if (more) lm_copy_wait<1>(); else lm_copy_wait<0>();
         __syncthreads();                                  // every thread's copies of this tile (and the queries) are in place
@@ -159,7 +162,7 @@ latent_attn_mma_kernel(const LatentArgs a) {
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const int key = k0 + 8 * j + 2 * t4 + (i & 1);
-                s[j][i] = key <= k_last ? s[j][i] : -INFINITY;
+                s[j][i] = key <= k_last && key >= first ? s[j][i] : -INFINITY;
                 mx[i >> 1] = fmaxf(mx[i >> 1], s[j][i]);
             }
         float alpha[2], m_use[2];
@@ -230,7 +233,7 @@ latent_attn_mma_kernel(const LatentArgs a) {
                 }
         } else {
             const float gt = a.gate ? sigmoid_f32(to_f32(((const bf16*)a.gate)[t * a.ld_gate + h])) : 1.f;
-            const float f = gt / l_run[half];
+            const float f = gt / (l_run[half] + (a.sink ? exp2f(a.sink[h] * 1.4426950408889634f - m_run[half]) : 0.f));
             float* out = a.out + t * a.ldo + (long long)h * KR;
 #pragma unroll
             for (int j = 0; j < NT; ++j)
@@ -249,6 +252,7 @@ extern "C" int cm_latent_attn_mma(const LatentArgs* args, cudaStream_t st) {
     if (a.rows <= 0 || a.B <= 0) return CM_OK;
     if (a.E != a.KR + a.R || a.KR < 1 || a.KR > 512 || a.EC % 8 || a.EC < a.E || ((uintptr_t)a.pool & 15))
         CM_REFUSE("latent_attn_mma: latents of %d channels (up to 512) in entries of %d (a multiple of 8, 16-byte aligned)", a.KR, a.EC);
+    if (a.ckv || a.ring % PAGE_TOKENS) CM_REFUSE("latent_attn_mma: reads the cache only, a ring of whole pages");
     if (a.splits < 1 || (a.splits > 1 && (!a.parts || a.chunk < LM_KT || a.chunk % LM_KT)))
         CM_REFUSE("latent_attn_mma: %d splits of %d keys", a.splits, a.chunk);
     const int nt = a.KR <= 128 ? 4 : (a.KR <= 256 ? 8 : 16);

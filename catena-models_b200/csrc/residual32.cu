@@ -134,6 +134,105 @@ postnorm_residual_kernel(float* __restrict__ h, T* __restrict__ n_out, ResidualT
     }
 }
 
+// The norm on what is added: h += norm(terms) * w.  n_out <- T(h) when given, or with w_next T(norm(h) * w_next): the rows
+// as the next reader takes them.
+template <typename T>
+__global__ void __launch_bounds__(R32_THREADS)
+outnorm_residual_kernel(float* __restrict__ h, T* __restrict__ n_out, ResidualTerms terms, const float* __restrict__ w,
+                        const float* __restrict__ w_next, int H, float eps, float eps_next) {
+    extern __shared__ float row[];
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const long long r = blockIdx.x;
+    float* hr = h + r * H;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < H; c += R32_THREADS) {
+        const float v = terms_at<T>(terms, r, H, c);
+        row[c] = v;
+        ss += v * v;
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)H + eps);
+    float hs = 0.f;
+    for (int c = threadIdx.x; c < H; c += R32_THREADS) {     // every thread reads back what it stored itself
+        const float x = fmaf(row[c] * inv, w[c], hr[c]);
+        hr[c] = x;
+        row[c] = x;
+        hs += x * x;
+        if (n_out && !w_next) n_out[r * H + c] = from_f32<T>(x);
+    }
+    if (!n_out || !w_next) return;
+    hs = block_sum(hs, scratch);
+    const float inv_next = 1.f / sqrtf(hs / (float)H + eps_next);
+    for (int c = threadIdx.x; c < H; c += R32_THREADS) n_out[r * H + c] = from_f32<T>((row[c] * inv_next) * w_next[c]);
+}
+
+// The same with 16-byte accesses for terms that are plain rows (one piece a row, or one row for all): a thread owns four
+// consecutive columns at a time and keeps them in registers.
+#define R32_VEC_MAX 8              // chunks of 4 * R32_THREADS columns: rows of up to 8,192
+template <typename T>
+__device__ __forceinline__ float4 term4(const ResidualTerm& t, long long i) {
+    if (t.is_f32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(t.p) + i);
+    const T* p = reinterpret_cast<const T*>(t.p) + i;
+    return make_float4(to_f32(p[0]), to_f32(p[1]), to_f32(p[2]), to_f32(p[3]));
+}
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(bf16* p, float4 v) {
+    __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+    *reinterpret_cast<uint2*>(p) = *reinterpret_cast<uint2*>(h);
+}
+template <typename T, int CH>
+__global__ void __launch_bounds__(R32_THREADS)
+outnorm_residual_vec_kernel(float* __restrict__ h, T* __restrict__ n_out, ResidualTerms terms, const float* __restrict__ w,
+                            const float* __restrict__ w_next, int H, float eps, float eps_next) {
+    __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
+    const long long r = blockIdx.x;
+    float* hr = h + r * H;
+    float4 y[CH], x[CH];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < CH; ++k) {
+        const int c = (k * R32_THREADS + threadIdx.x) * 4;
+        y[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c >= H) continue;
+        x[k] = *reinterpret_cast<const float4*>(hr + c);
+        for (int i = 0; i < terms.n; ++i) {
+            const ResidualTerm& t = terms.t[i];
+            const float4 v = term4<T>(t, (t.per_row ? r * H : 0) + c);
+            y[k].x += t.scale * v.x; y[k].y += t.scale * v.y; y[k].z += t.scale * v.z; y[k].w += t.scale * v.w;
+        }
+        ss += y[k].x * y[k].x + y[k].y * y[k].y + y[k].z * y[k].z + y[k].w * y[k].w;
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.f / sqrtf(ss / (float)H + eps);
+    float hs = 0.f;
+#pragma unroll
+    for (int k = 0; k < CH; ++k) {
+        const int c = (k * R32_THREADS + threadIdx.x) * 4;
+        if (c >= H) continue;
+        const float4 wv = *reinterpret_cast<const float4*>(w + c);
+        x[k].x = fmaf(y[k].x * inv, wv.x, x[k].x); x[k].y = fmaf(y[k].y * inv, wv.y, x[k].y);
+        x[k].z = fmaf(y[k].z * inv, wv.z, x[k].z); x[k].w = fmaf(y[k].w * inv, wv.w, x[k].w);
+        put4(hr + c, x[k]);
+        hs += x[k].x * x[k].x + x[k].y * x[k].y + x[k].z * x[k].z + x[k].w * x[k].w;
+        if (n_out && !w_next) put4(n_out + r * H + c, x[k]);
+    }
+    if (!n_out || !w_next) return;
+    hs = block_sum(hs, scratch);
+    const float inv_next = 1.f / sqrtf(hs / (float)H + eps_next);
+#pragma unroll
+    for (int k = 0; k < CH; ++k) {
+        const int c = (k * R32_THREADS + threadIdx.x) * 4;
+        if (c >= H) continue;
+        const float4 wv = *reinterpret_cast<const float4*>(w_next + c);
+        put4(n_out + r * H + c, make_float4((x[k].x * inv_next) * wv.x, (x[k].y * inv_next) * wv.y, (x[k].z * inv_next) * wv.z,
+                                            (x[k].w * inv_next) * wv.w));
+    }
+}
+
 // out[r] = T([a[r]; b[r]]) for float rows a and b of width H: the input of a projection over both.
 template <typename T>
 __global__ void concat_cast_kernel(T* __restrict__ out, const float* __restrict__ a, const float* __restrict__ b,
@@ -225,6 +324,43 @@ extern "C" int cm_postnorm_residual(int dt, float* h, void* n_out, int n_terms, 
         return CM_ERR_DTYPE;
     CM_CHECK_LAUNCH();
     return CM_OK;
+}
+
+// The sum with the norm on what is added (outnorm_residual_kernel); terms as for cm_residual_add_norm.
+template <typename T>
+static int launch_outnorm(float* h, void* n_out, const ResidualTerms& terms, const float* w, const float* w_next, int rows, int H,
+                          float eps, float eps_next, size_t smem, cudaStream_t st) {
+    bool vec = H % 4 == 0 && H <= 4 * R32_THREADS * R32_VEC_MAX &&
+               (((uintptr_t)h | (uintptr_t)w | (uintptr_t)w_next) & 15) == 0 && ((uintptr_t)n_out & (4 * sizeof(T) - 1)) == 0;
+    for (int i = 0; i < terms.n; ++i)
+        vec = vec && terms.t[i].per_row <= 1 && !terms.t[i].index && !terms.t[i].weights && ((uintptr_t)terms.t[i].p & 15) == 0;
+    if (vec) {
+        const int ch = (H + 4 * R32_THREADS - 1) / (4 * R32_THREADS);
+#define ON_CASE(C) cm_launch(outnorm_residual_vec_kernel<T, C>, rows, R32_THREADS, 0, st, h, (T*)n_out, terms, w, w_next, H, eps, eps_next)
+        if (ch <= 1) ON_CASE(1); else if (ch <= 2) ON_CASE(2); else if (ch <= 4) ON_CASE(4); else ON_CASE(8);
+#undef ON_CASE
+    } else {
+        if (smem > 48 * 1024) cudaFuncSetAttribute(outnorm_residual_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cm_launch(outnorm_residual_kernel<T>, rows, R32_THREADS, smem, st, h, (T*)n_out, terms, w, w_next, H, eps, eps_next);
+    }
+    CM_CHECK_LAUNCH();
+    return CM_OK;
+}
+
+extern "C" int cm_outnorm_residual(int dt, float* h, void* n_out, int n_terms, const void* const* term_ptr,
+                                   const float* term_scale, const int* term_per_row, const int* term_is_f32,
+                                   const int* const* term_index, const float* const* term_weights, const float* w,
+                                   const float* w_next, int rows, int H, float eps, float eps_next, cudaStream_t st) {
+    if (rows <= 0) return CM_OK;
+    if (n_terms < 1 || n_terms > R32_MAX_TERMS) CM_REFUSE("outnorm_residual: %d terms (1 to %d)", n_terms, R32_MAX_TERMS);
+    if (!w || (w_next && !n_out)) CM_REFUSE("outnorm_residual: a norm needs its weight, and the next reader's norm a place for its rows");
+    size_t smem;
+    if (row_smem(H, &smem) != CM_OK) return CM_ERR_SHAPE;
+    ResidualTerms terms;
+    fill_terms(terms, n_terms, term_ptr, term_scale, term_per_row, term_is_f32, term_index, term_weights);
+    if (dt == DT_F32) return launch_outnorm<float>(h, n_out, terms, w, w_next, rows, H, eps, eps_next, smem, st);
+    if (dt == DT_BF16) return launch_outnorm<bf16>(h, n_out, terms, w, w_next, rows, H, eps, eps_next, smem, st);
+    return CM_ERR_DTYPE;
 }
 
 extern "C" int cm_concat_cast(int dt, void* out, const float* a, const float* b, long long rows, int H, cudaStream_t st) {

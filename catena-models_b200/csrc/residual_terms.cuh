@@ -11,7 +11,7 @@ struct ResidualTerm {
     const int* index;      // null: piece j of row r is row r * per_row + j; else row index[r * per_row + j] (negative: none)
     const float* weights;  // null, or a factor per piece: weights[r * per_row + j] (a routed feed-forward's weights on its experts' outputs)
     float scale;
-    int per_row;
+    int per_row;           // 0: one row that is added to every row (a bias)
     int is_f32;
 };
 struct ResidualTerms {
@@ -30,7 +30,7 @@ __device__ __forceinline__ float terms_at(const ResidualTerms& terms, long long 
     float add = 0.f;
     for (int i = 0; i < terms.n; ++i) {
         const ResidualTerm& t = terms.t[i];
-        float s = 0.f;
+        float s = t.per_row ? 0.f : term_at<T>(t, c);
         for (int j = 0; j < t.per_row; ++j) {
             const long long piece = t.index ? t.index[r * t.per_row + j] : r * t.per_row + j;
             if (piece >= 0) {

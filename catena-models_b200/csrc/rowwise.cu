@@ -404,23 +404,23 @@ extern "C" int cm_swiglu(int dt, void* a, const void* gu, int rows, int F, int a
     return CM_OK;
 }
 
-// ------------------------------------------------------------ squared ReLU
-// x <- T(max(x, 0)^2) in place: the activation between the two products of a plain feed-forward.
+// ------------------------------------------------------------ activations of a plain feed-forward
+// x <- T(act(x)) in place, between the two products: kind 0 max(x, 0)^2, kind 1 the tanh form of gelu.
 template <typename T>
-__global__ void relu2_kernel(T* __restrict__ x, long long total) {
+__global__ void act_inplace_kernel(T* __restrict__ x, long long total, int kind) {
     pdl_trigger();
     pdl_wait();
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
-        const float v = fmaxf(to_f32(x[i]), 0.f);
-        x[i] = from_f32<T>(v * v);
+        const float z = to_f32(x[i]), v = fmaxf(z, 0.f);
+        x[i] = from_f32<T>(kind == 1 ? gelu_tanh_f32(z) : v * v);
     }
 }
 
-extern "C" int cm_relu2_inplace(int dt, void* x, long long total, cudaStream_t st) {
+extern "C" int cm_act_inplace(int dt, void* x, long long total, int kind, cudaStream_t st) {
     if (total <= 0) return CM_OK;
     const unsigned blocks = (unsigned)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
-    if (dt == DT_F32) cm_launch(relu2_kernel<float>, blocks, 256, 0, st, (float*)x, total);
-    else if (dt == DT_BF16) cm_launch(relu2_kernel<bf16>, blocks, 256, 0, st, (bf16*)x, total);
+    if (dt == DT_F32) cm_launch(act_inplace_kernel<float>, blocks, 256, 0, st, (float*)x, total, kind);
+    else if (dt == DT_BF16) cm_launch(act_inplace_kernel<bf16>, blocks, 256, 0, st, (bf16*)x, total, kind);
     else return CM_ERR_DTYPE;
     CM_CHECK_LAUNCH();
     return CM_OK;

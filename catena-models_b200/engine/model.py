@@ -135,6 +135,12 @@ class DecoderModel:
             h, n = first_norm.open(rt, h)
         elif first_norm is not None:
             n = first_norm.apply(rt, h)
+        elif n is None and self.blocks[plan[0].block].reads_stream:
+            n = h
+            if h.dtype != rt.dtype:
+                n = torch.empty(h.shape, dtype=rt.dtype, device=rt.device)
+                kernels.embed_gather(n, self.embedding, batch.tokens, self.token_error, sampled=batch.prev_sampled,
+                                     scale=self.definition.embedding_scale)
         # when every row is wanted in order (a decode step), the last block's fused residual kernel
         # applies the final norm too and no rows need gathering
         whole = batch.wants_every_row and batch.n_want == batch.T

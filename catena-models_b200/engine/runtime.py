@@ -289,12 +289,36 @@ class Runtime:
         kernels.swiglu(a, gu, act=flag - 1 if flag is not True else 0, limit=limit)
         return a
 
+    def linear_gelu(self, x, w):
+        """a = gelu(x @ w^T), the tanh form, in x's dtype: in the epilogue of the tensor-core and streaming products."""
+        kind = self._product_kernel(x, w)
+        if kind == "skinny" and 8 < x.shape[0] <= self.SKINNY_BEST_ROWS and w.shape[1] >= 2048 and self._tma_operands(x, w):
+            kind = "few_rows"                              # as for a plain product (`linear`)
+        a = torch.empty((x.shape[0], w.shape[0]), dtype=x.dtype, device=x.device)
+        if kind == "skinny":
+            kernels.gemm_skinny(a, x, w, swiglu=kernels.GATE_GELU)
+        elif kind == "few_rows":
+            kernels.gemm_tc_few_rows(a, x, w, swiglu=kernels.GATE_GELU, err=self.error_flag)
+        elif kind == "tiled":
+            kernels.gemm_tc(a, x, w, swiglu=kernels.GATE_GELU, err=self.error_flag, block_n=self._tile_width(x.shape[0], w.shape[0]))
+        else:
+            kernels.gemm_simt(a, x, w)
+            kernels.act_inplace(a, "gelu_tanh")
+        return a
+
     # ------------------------------------------------------------------ attention
     TCGEN05_ATTENTION_MIN_LEN = 768      # shorter prompts (or windows) give an item too few key tiles to pipeline ...
     TCGEN05_ATTENTION_MIN_LEN_BATCH = 256    # ... unless there are many of them:
     TCGEN05_ATTENTION_MIN_TOKENS = 2048      # this many rows in the step
 
-    def attention_prefill(self, ctx, q, k, v, gate, batch, QH, KVH, HD, window, scale, sink=None, softcap=0.0):
+    @staticmethod
+    def _stores(width, HD, value_dim, gate, gate_channels):
+        """True if an attention kernel that stores `width` channels at a time can leave `value_dim` of HD, gated per channel."""
+        return (value_dim or HD) % width == 0 and not (
+            gate_channels and (gate.stride(0) % width or gate.data_ptr() % (2 * width)))
+
+    def attention_prefill(self, ctx, q, k, v, gate, batch, QH, KVH, HD, window, scale, sink=None, softcap=0.0, value_dim=None,
+                          gate_channels=False):
         """Attention of a prompt step over the step's own keys and values.  bfloat16 with head size
         64 or 128 and long sequences: the tcgen05 kernel (measured on B200, 32 heads of 64, tcgen05 against
         mma.sync: 18 / 25 us at 768 tokens, 22 / 35 at 1,024, 40 / 96 at 2,048, 664 against 264 TFLOP/s at
@@ -310,12 +334,16 @@ class Runtime:
         long_enough = span >= self.TCGEN05_ATTENTION_MIN_LEN or (
             span >= self.TCGEN05_ATTENTION_MIN_LEN_BATCH and q.shape[0] >= self.TCGEN05_ATTENTION_MIN_TOKENS)
         if (bf16 and aligned and HD in (64, 128) and long_enough
-                and ctx.stride(0) % 8 == 0 and ctx.data_ptr() % 16 == 0):
+                and ctx.stride(0) % 8 == 0 and ctx.data_ptr() % 16 == 0
+                and self._stores(8, HD, value_dim, gate, gate_channels)):
             kernels.attn_prefill_tc(ctx, q, k, v, gate, batch.seq_start, batch.B, batch.max_len, QH, KVH, HD, window,
-                                    scale, err=self.error_flag, sink=sink, softcap=softcap)
+                                    scale, err=self.error_flag, sink=sink, softcap=softcap, value_dim=value_dim,
+                                    gate_channels=gate_channels)
             return
-        fn = kernels.attn_prefill_mma if (bf16 and aligned and HD % 16 == 0 and HD <= 128) else kernels.attn_prefill_simt
-        fn(ctx, q, k, v, gate, batch.seq_start, batch.B, batch.max_len, QH, KVH, HD, window, scale, sink=sink, softcap=softcap)
+        mma = bf16 and aligned and HD % 16 == 0 and HD <= 128 and ctx.stride(0) % 2 == 0 and self._stores(2, HD, value_dim, gate, gate_channels)
+        fn = kernels.attn_prefill_mma if mma else kernels.attn_prefill_simt
+        fn(ctx, q, k, v, gate, batch.seq_start, batch.B, batch.max_len, QH, KVH, HD, window, scale, sink=sink, softcap=softcap,
+           value_dim=value_dim, gate_channels=gate_channels)
 
     # Measured on B200, 32 heads of 64 over 8 kv heads, mma.sync against tcgen05:
     # 128 rows on 512 held tokens 20.9 / 17.0 us, on 256 held 13.4 / 13.3; 64 rows on 256 held 12.1 / 13.2; 16 rows x 8
@@ -324,7 +352,8 @@ class Runtime:
     TCGEN05_APPEND_MIN_ROWS = 8
     TCGEN05_APPEND_MIN_SPAN = 512
 
-    def attention_append(self, ctx, q, k, v, gate, batch, state, QH, KVH, HD, window, scale, sink=None, softcap=0.0):
+    def attention_append(self, ctx, q, k, v, gate, batch, state, QH, KVH, HD, window, scale, sink=None, softcap=0.0, value_dim=None,
+                         gate_channels=False):
         """Attention of a step whose sequences already hold tokens: keys and values below each
         sequence's first position of the step come from the paged cache, the rest from the step's own
         rows (written to the cache by the caller afterwards).  The choice of kernel follows
@@ -336,11 +365,14 @@ class Runtime:
         bf16 = q.dtype == torch.bfloat16 and state.pool.dtype == torch.bfloat16 and self.tensor_core_prompts
         span = min(batch.max_end, abs(window)) if window else batch.max_end
         if (bf16 and aligned and HD in (64, 128) and span >= self.TCGEN05_APPEND_MIN_SPAN
-                and batch.max_len >= self.TCGEN05_APPEND_MIN_ROWS and ctx.stride(0) % 8 == 0 and ctx.data_ptr() % 16 == 0):
+                and batch.max_len >= self.TCGEN05_APPEND_MIN_ROWS and ctx.stride(0) % 8 == 0 and ctx.data_ptr() % 16 == 0
+                and self._stores(8, HD, value_dim, gate, gate_channels)):
             kernels.attn_append_tc(ctx, q, k, v, gate, batch.seq_start, batch.seq_pos0, batch.seq_slot, state.pool,
                                    state.pages, state.ptab, state.ring, batch.B, batch.max_len, QH, KVH, HD, window,
-                                   scale, err=self.error_flag, sink=sink, softcap=softcap)
+                                   scale, err=self.error_flag, sink=sink, softcap=softcap, value_dim=value_dim,
+                                   gate_channels=gate_channels)
             return
         kernels.attn_append(ctx, q, k, v, gate, batch.seq_start, batch.seq_pos0, batch.seq_slot, state.pool,
                             state.pages, state.ptab, state.ring, batch.B, batch.max_len, QH, KVH, HD, window, scale,
-                            tensor_cores=self.tensor_core_prompts, sink=sink, softcap=softcap)
+                            tensor_cores=self.tensor_core_prompts, sink=sink, softcap=softcap, value_dim=value_dim,
+                            gate_channels=gate_channels)

@@ -34,19 +34,19 @@ _SIGNATURES = {
     "cm_gemm_tc_few_rows": [_i, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _f, _vp],
     "cm_qk_prepare": [_i, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _i,
                       _i, _i, _f, _i, _f, _i, _vp],
-    "cm_attn_prefill_simt": [_i, _vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp],
-    "cm_attn_prefill_mma": [_vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp],
-    "cm_attn_prefill_tc": [_vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _ll, _i, _i, _i, _i, _f, _f, _vp, _vp, _vp],
+    "cm_attn_prefill_simt": [_i, _vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _i, _i, _vp],
+    "cm_attn_prefill_mma": [_vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _i, _i, _vp],
+    "cm_attn_prefill_tc": [_vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _i, _ll, _i, _i, _i, _i, _f, _f, _vp, _i, _i, _vp, _vp],
     "cm_attn_decode": [_i, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _i, _i, _i,
-                       _i, _f, _f, _vp, _vp, _vp, _vp],
+                       _i, _f, _f, _vp, _vp, _vp, _i, _i, _vp],
     "cm_gemm_skinny_shortconv": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _ll, _ll, _ll, _vp],
     "cm_shortconv": [_i, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "cm_attn_append_simt": [_i, _vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _i, _i, _i,
-                            _i, _i, _i, _f, _f, _vp, _vp],
+                            _i, _i, _i, _f, _f, _vp, _i, _i, _vp],
     "cm_attn_append_mma": [_vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _i, _i, _i, _i,
-                           _i, _i, _f, _f, _vp, _vp],
+                           _i, _i, _f, _f, _vp, _i, _i, _vp],
     "cm_attn_append_tc": [_vp, _ll, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _i, _i, _ll, _i,
-                          _i, _i, _i, _f, _f, _vp, _vp, _vp],
+                          _i, _i, _i, _f, _f, _vp, _i, _i, _vp, _vp],
     "cm_gemm_tc_parts": [_vp, _vp, _vp, _i, _i, _i, _ll, _ll, _i, _i, _vp, _vp],
     "cm_kv_store": [_i, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _i, _i, _i, _i, _vp],
     "cm_sample": [_vp, _vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp],
@@ -59,7 +59,9 @@ _SIGNATURES = {
     "cm_hyper_connect": [_i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _f, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "cm_delta_prompt": [_i, _vp, _vp],
     "cm_delta_step": [_i, _vp, _vp],
-    "cm_relu2_inplace": [_i, _vp, _ll, _vp],
+    "cm_outnorm_residual": [_i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _f, _vp],
+    "cm_head_prepare": [_i, _vp, _vp],
+    "cm_act_inplace": [_i, _vp, _ll, _i, _vp],
     "cm_tap_rotate_store": [_i, _vp, _vp],
     "cm_diff_attn": [_i, _vp, _i, _i, _vp, _i, _vp],
     "cm_diff_attn_mma": [_vp, _i, _vp],
@@ -74,11 +76,12 @@ _SIGNATURES = {
     "cm_moe_route": [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _i, _i, _i, _f, _f, _i, _vp, _vp],
     "cm_moe_identity": [_i, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _vp],
     "cm_latent_prepare": [_i, _vp, _vp],
+    "cm_latent_store": [_i, _vp, _vp],
     "cm_latent_query_turn": [_i, _vp, _vp],
     "cm_latent_expand": [_i, _vp, _vp],
     "cm_latent_attn": [_i, _vp, _vp],
     "cm_latent_attn_mma": [_vp, _vp],
-    "cm_head_linear": [_i, _vp, _vp, _vp, _ll, _i, _i, _i, _ll, _ll, _i, _i, _i, _i, _vp],
+    "cm_head_linear": [_i, _vp, _vp, _vp, _ll, _i, _i, _i, _ll, _ll, _i, _i, _i, _i, _vp, _ll, _vp],
     "cm_moe_gather": [_i, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _vp],
     "cm_gemm_tc_grouped": [_i, _vp, _vp, _vp, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _i, _vp, _f, _vp],
     "cm_moe_grouped": [_i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
@@ -365,7 +368,8 @@ class PartialSums:
 class Terms(list):
     """What a sublayer adds to a float32 residual stream: (tensor, factor, pieces per row[, index[, weights]])
     entries; the tensor holds a row's pieces one below the other (rows * pieces rows), or anywhere, with `index`
-    (int32 [rows * pieces], negative: no piece) saying where; `weights` (float32 [rows * pieces]): a factor on
+    (int32 [rows * pieces], negative: no piece) saying where; 0 pieces: the tensor is one row that is added to every row (a
+    bias); `weights` (float32 [rows * pieces]): a factor on
     each piece; float32 or the activation dtype (`residual_add_norm`, `postnorm_residual`)."""
 
 
@@ -447,18 +451,24 @@ def gemm_simt(y, x, w):
            cost=lambda: (f"{M}x{N}x{K}", _nbytes(x, w, y), 2 * M * N * K))
 
 
-_GATE_SUFFIX = ("", "_swiglu", "_geglu", "_clamped")     # a product's name by its gate flag
+_GATE_SUFFIX = ("", "_swiglu", "_geglu", "_clamped", "_gelu")     # a product's name by its gate flag
+GATE_GELU = 4                       # the flag of the form without a gate: the tanh form of gelu on every output
+
+
+def _gated(flag):
+    """True if a product with this flag takes the packed rows [gate; up]."""
+    return bool(flag) and int(flag) != GATE_GELU
 
 
 def gemm_skinny(y, x, w, swiglu=False, limit=0.0):
     """y = x @ w^T for at most 64 bfloat16 rows, weights streamed once (mma.sync, float sums).
     swiglu: w is [gate; up] with 2F rows and y[M, F] = silu(x Wgate^T) * (x Wup^T); swiglu=2 (all products that
     take the flag): the tanh form of gelu in silu's place; swiglu=3 with `limit` L: the clamped gate, g' sigmoid(1.702 g')
-    (u' + 1) with g' = min(g, L), u' = clamp(u, -L, L)."""
+    (u' + 1) with g' = min(g, L), u' = clamp(u, -L, L); swiglu=4: no gate, the tanh form of gelu on every output (w [N, K])."""
     _need_cuda(y, x, w)
     M, K = x.shape
     N = y.shape[1]
-    if w.shape[1] != K or w.shape[0] != (2 * N if swiglu else N) or y.shape[0] != M:
+    if w.shape[1] != K or w.shape[0] != (2 * N if _gated(swiglu) else N) or y.shape[0] != M:
         raise KernelError(f"gemm_skinny shapes: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("gemm_skinny takes bfloat16 operands")
@@ -533,7 +543,7 @@ def gemm_tc(y, x, w, swiglu=False, err=None, block_n=256, limit=0.0):
     _need_cuda(y, x, w)
     M, K = x.shape
     N = y.shape[1]
-    if w.shape[1] != K or w.shape[0] != (2 * N if swiglu else N) or y.shape[0] != M:
+    if w.shape[1] != K or w.shape[0] != (2 * N if _gated(swiglu) else N) or y.shape[0] != M:
         raise KernelError(f"gemm_tc shapes: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("gemm_tc takes bfloat16 operands")
@@ -551,7 +561,7 @@ def gemm_tc_few_rows(y, x, w, swiglu=False, err=None, splits=0, limit=0.0):
     _need_cuda(y, x, w)
     M, K = x.shape
     N = y.shape[1]
-    if w.shape[1] != K or w.shape[0] != (2 * N if swiglu else N) or y.shape[0] != M:
+    if w.shape[1] != K or w.shape[0] != (2 * N if _gated(swiglu) else N) or y.shape[0] != M:
         raise KernelError(f"gemm_tc_few_rows shapes: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("gemm_tc_few_rows takes bfloat16 operands")
@@ -581,45 +591,92 @@ def qk_prepare(qkv, wq, wk, rate, tok_pos, tok_seq, seq_slot, seq_end, pool, pag
                          T * HD * qkv.element_size() * (2 * QH + (2 * KVH if pool is None else 4 * KVH)), 0))
 
 
-def attn_prefill_simt(ctx, q, k, v, gate, seq_start, B, max_len, QH, KVH, HD, window, scale, sink=None, softcap=0.0):
+class _HeadPrepareArgs(ctypes.Structure):
+    """csrc/head_prepare.h: HeadPrepareArgs."""
+    _fields_ = [("qkv", _vp), ("ld", _ll), ("bias", _vp), ("wq", _vp), ("wk", _vp), ("rate", _vp), ("v_first", _vp), ("ld_first", _ll),
+                ("lam", _vp), ("tok_pos", _vp), ("tok_seq", _vp), ("seq_slot", _vp), ("seq_end", _vp), ("pool", _vp), ("pages", _ll),
+                ("ptab", _vp), ("ptab_stride", _ll), ("rows", _ll)] \
+        + [(n, _i) for n in ("QH", "KVH", "HD", "norm_dim", "pairs", "interleaved", "ring", "DV", "DV1", "HD1", "vec_first")] \
+        + [("eps", _f), ("mag", _f)]
+
+
+def head_prepare(qkv, batch, QH, KVH, HD, bias=None, wq=None, wk=None, norm_dim=None, eps=0.0, rate=None, interleaved=False, mag=1.0,
+                 value_dim=None, mix=None, kv=None):
+    """Everything between an attention layer's packed projection rows [q | k | v | ...] and its attention kernel, in place:
+    `bias` (float32 [(QH + 2 KVH) HD]); a norm per query and key head (`wq`, `wk` float32 [HD] or None, the mean of squares over
+    `norm_dim` channels); the rotation of q and k by position * rate[i] for the leading rate.numel() pairs (neighbours with
+    `interleaved`, else channel i with i + HD / 2), `mag` the factor on sine and cosine; `mix` = (values, their channels a head
+    without and with padding, share): v <- (1 - share) v + share values, channel by channel of the unpadded value rows (share: one
+    float32 on the device; values: a view of rows in qkv's dtype).  `value_dim`: this layer's value channels a head without
+    padding.  `kv` = (pool, pages, ptab, ring): k and v also go to the cache.  Between load and store all is float32."""
+    rows = qkv.shape[0]
+    if qkv.stride(1) != 1 or qkv.shape[1] < (QH + 2 * KVH) * HD:
+        raise KernelError("head_prepare: rows [q | k | v | ...]")
+    for t, n in ((bias, (QH + 2 * KVH) * HD), (wq, HD), (wk, HD), (rate, None)):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or (n is not None and t.numel() != n)):
+            raise KernelError("head_prepare: float32 constants of the heads' sizes")
+    value_dim = value_dim or HD
+    first, dv1, hd1, lam = mix if mix is not None else (None, 0, 0, None)
+    if first is not None and (first.dtype != qkv.dtype or first.shape[0] != rows or first.stride(1) != 1 or lam.dtype != torch.float32
+                              or (KVH * value_dim - 1) // dv1 * hd1 + (KVH * value_dim - 1) % dv1 >= first.shape[1]):
+        raise KernelError("head_prepare: the values to mix in do not cover this layer's")
+    pool, pages, ptab, ring = kv if kv is not None else (None, 0, None, 0)
+    a = _HeadPrepareArgs(qkv=_ptr(qkv), ld=qkv.stride(0), bias=_ptr(bias), wq=_ptr(wq), wk=_ptr(wk), rate=_ptr(rate), v_first=_ptr(first),
+                         ld_first=0 if first is None else first.stride(0), lam=_ptr(lam), tok_pos=_ptr(batch.tok_pos),
+                         tok_seq=_ptr(batch.tok_seq), seq_slot=_ptr(batch.seq_slot), seq_end=_ptr(batch.seq_end), pool=_ptr(pool),
+                         pages=pages, ptab=_ptr(ptab), ptab_stride=0 if ptab is None else ptab.stride(0), rows=rows, QH=QH, KVH=KVH,
+                         HD=HD, norm_dim=norm_dim or HD, pairs=0 if rate is None else rate.numel(), interleaved=int(interleaved),
+                         ring=ring, DV=value_dim, DV1=dv1, HD1=hd1, eps=eps, mag=mag)
+    _check(lib().cm_head_prepare(dtype_code(qkv.dtype), ctypes.byref(a), _stream()), "head_prepare",
+           cost=lambda: (f"{rows} tokens, {QH}+{KVH}+{KVH} heads of {HD}",
+                         rows * HD * qkv.element_size() * (2 * (QH + 2 * KVH) + (2 * KVH if pool is not None else 0) + (KVH if first is not None else 0)), 0))
+
+
+def attn_prefill_simt(ctx, q, k, v, gate, seq_start, B, max_len, QH, KVH, HD, window, scale, sink=None, softcap=0.0, value_dim=None,
+                      gate_channels=False):
     """q, k, v, gate are column views of one packed row-major buffer (same row stride).  `sink` (all
     attention kernels): float32 [QH], a learned logit per query head that joins the softmax's denominator
     and nothing else (it has no key and no value), or None.  `softcap` (all attention kernels) = c > 0: every
     score is bounded before the mask and the softmax, s <- c * tanh(s / c) with s = (q . k) * scale.  `window` (all
     attention kernels): W > 0, a query sees the last W positions; W < 0, the positions of its own chunk, chunks of -W
-    positions counted from the sequence's start; 0, every earlier position."""
+    positions counted from the sequence's start; 0, every earlier position.  `value_dim` (all attention kernels): how many
+    of a head's HD value channels are stored, the heads side by side in ctx's rows (default all; the rest is padding).
+    `gate_channels` (all attention kernels): `gate` holds a logit per stored channel, [rows, >= QH * value_dim], instead of
+    one per head."""
     if not (q.stride(0) == k.stride(0) == v.stride(0)):
         raise KernelError("attn_prefill: q, k and v must share a row stride")
     _check(lib().cm_attn_prefill_simt(dtype_code(q.dtype), _ptr(ctx), ctx.stride(0), _ptr(q), _ptr(k), _ptr(v),
                                       q.stride(0), _ptr(gate), 0 if gate is None else gate.stride(0),
-                                      _ptr(seq_start), B, max_len, QH, KVH, HD, window, scale, softcap, _ptr(sink), _stream()),
-           "attn_prefill_simt",
+                                      _ptr(seq_start), B, max_len, QH, KVH, HD, window, scale, softcap, _ptr(sink), value_dim or HD, int(gate_channels),
+                                      _stream()), "attn_prefill_simt",
            cost=lambda: (f"{B} sequences up to {max_len}, {QH}/{KVH} heads of {HD}, window {window}", 0, 0))
 
 
-def attn_prefill_mma(ctx, q, k, v, gate, seq_start, B, max_len, QH, KVH, HD, window, scale, sink=None, softcap=0.0):
+def attn_prefill_mma(ctx, q, k, v, gate, seq_start, B, max_len, QH, KVH, HD, window, scale, sink=None, softcap=0.0, value_dim=None,
+                      gate_channels=False):
     """The same on the tensor cores: bfloat16, head sizes that are multiples of 16 up to 128."""
     if not (q.stride(0) == k.stride(0) == v.stride(0)) or q.dtype != torch.bfloat16:
         raise KernelError("attn_prefill_mma: bfloat16 q, k and v that share a row stride")
     _check(lib().cm_attn_prefill_mma(_ptr(ctx), ctx.stride(0), _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(gate),
                                      0 if gate is None else gate.stride(0), _ptr(seq_start), B, max_len, QH, KVH,
-                                     HD, window, scale, softcap, _ptr(sink), _stream()), "attn_prefill_mma",
+                                     HD, window, scale, softcap, _ptr(sink), value_dim or HD, int(gate_channels), _stream()), "attn_prefill_mma",
            cost=lambda: (f"{B} sequences up to {max_len}, {QH}/{KVH} heads of {HD}, window {window}", 0, 0))
 
 
 def attn_append(ctx, q, k, v, gate, seq_start, seq_pos0, seq_slot, pool, pages, ptab, ring, B, max_len, QH, KVH, HD,
-                window, scale, tensor_cores=True, sink=None, softcap=0.0):
+                window, scale, tensor_cores=True, sink=None, softcap=0.0, value_dim=None, gate_channels=False):
     """Attention of a step whose sequences may stand at seq_pos0[b] > 0: keys and values below that
     position come from the paged cache `pool`, the rest from the step's own rows (q, k, v as for the
     prefill kernels), which the caller writes to the cache afterwards (`kv_store`).  bfloat16 with a
     head size that is a multiple of 16 up to 128 runs on the tensor cores unless `tensor_cores` is off."""
     if not (q.stride(0) == k.stride(0) == v.stride(0)):
         raise KernelError("attn_append: q, k and v must share a row stride")
-    mma = (tensor_cores and q.dtype == torch.bfloat16 and HD % 16 == 0 and HD <= 128 and q.stride(0) % 8 == 0
+    mma = (tensor_cores and q.dtype == torch.bfloat16 and HD % 16 == 0 and HD <= 128 and q.stride(0) % 8 == 0 and (value_dim or HD) % 2 == 0
+           and not (gate_channels and (gate.stride(0) % 2 or gate.data_ptr() % 4))
            and (q.data_ptr() | k.data_ptr() | v.data_ptr() | pool.data_ptr()) % 16 == 0)
     common = (_ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(seq_start),
               _ptr(seq_pos0), _ptr(seq_slot), _ptr(pool), pages, _ptr(ptab), ptab.stride(0), ring, B, max_len, QH, KVH,
-              HD, window, scale, softcap, _ptr(sink), _stream())
+              HD, window, scale, softcap, _ptr(sink), value_dim or HD, int(gate_channels), _stream())
     if mma:
         _check(lib().cm_attn_append_mma(_ptr(ctx), ctx.stride(0), *common), "attn_append_mma")
     else:
@@ -627,7 +684,7 @@ def attn_append(ctx, q, k, v, gate, seq_start, seq_pos0, seq_slot, pool, pages, 
 
 
 def attn_append_tc(ctx, q, k, v, gate, seq_start, seq_pos0, seq_slot, pool, pages, ptab, ring, B, max_len, QH, KVH, HD,
-                   window, scale, err=None, sink=None, softcap=0.0):
+                   window, scale, err=None, sink=None, softcap=0.0, value_dim=None, gate_channels=False):
     """`attn_append` on the tcgen05 tensor cores: bfloat16, head size 64 or 128, the cache read page by
     page with TMA.  err: device int32 that a block raises if a bounded pipeline wait runs out."""
     if (not (q.stride(0) == k.stride(0) == v.stride(0)) or q.dtype != torch.bfloat16 or pool.dtype != torch.bfloat16
@@ -638,7 +695,8 @@ def attn_append_tc(ctx, q, k, v, gate, seq_start, seq_pos0, seq_slot, pool, page
     _check(lib().cm_attn_append_tc(_ptr(ctx), ctx.stride(0), _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(gate),
                                    0 if gate is None else gate.stride(0), _ptr(seq_start), _ptr(seq_pos0),
                                    _ptr(seq_slot), _ptr(pool), pages, _ptr(ptab), ptab.stride(0), ring, B, max_len,
-                                   q.shape[0], QH, KVH, HD, window, scale, softcap, _ptr(sink), _ptr(err), _stream()), "attn_append_tc",
+                                   q.shape[0], QH, KVH, HD, window, scale, softcap, _ptr(sink), value_dim or HD, int(gate_channels), _ptr(err),
+                                   _stream()), "attn_append_tc",
            cost=lambda: (f"{B} sequences of up to {max_len} rows, {QH}/{KVH} heads of {HD}, window {window}", 0, 0))
 
 
@@ -651,7 +709,8 @@ def kv_store(kv, tok_pos, tok_seq, seq_slot, seq_end, pool, pages, ptab, ring, K
            "kv_store")
 
 
-def attn_prefill_tc(ctx, q, k, v, gate, seq_start, B, max_len, QH, KVH, HD, window, scale, err=None, sink=None, softcap=0.0):
+def attn_prefill_tc(ctx, q, k, v, gate, seq_start, B, max_len, QH, KVH, HD, window, scale, err=None, sink=None, softcap=0.0,
+                    value_dim=None, gate_channels=False):
     """The same on the tcgen05 tensor cores (TMA-fed, scores and outputs in tensor memory): bfloat16,
     head size 64 or 128.  q, k and v are column blocks of one row-major buffer.  err: device int32
     that a block raises if one of its bounded pipeline waits runs out."""
@@ -659,7 +718,8 @@ def attn_prefill_tc(ctx, q, k, v, gate, seq_start, B, max_len, QH, KVH, HD, wind
         raise KernelError("attn_prefill_tc: bfloat16 q, k and v that share rows and a row stride")
     _check(lib().cm_attn_prefill_tc(_ptr(ctx), ctx.stride(0), _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(gate),
                                     0 if gate is None else gate.stride(0), _ptr(seq_start), B, max_len, q.shape[0],
-                                    QH, KVH, HD, window, scale, softcap, _ptr(sink), _ptr(err), _stream()), "attn_prefill_tc",
+                                    QH, KVH, HD, window, scale, softcap, _ptr(sink), value_dim or HD, int(gate_channels), _ptr(err),
+                                    _stream()), "attn_prefill_tc",
            cost=lambda: (f"{B} sequences up to {max_len}, {QH}/{KVH} heads of {HD}, window {window}", 0, 0))
 
 
@@ -683,12 +743,12 @@ def attn_decode_scratch(B, QH, HD, n_chunks, device):
 
 
 def attn_decode(ctx, q, gate, seq_pos, seq_slot, pool, pages, ptab, ring, window, QH, KVH, HD, n_chunks,
-                scale, part_o, part_ml, sink=None, softcap=0.0):
+                scale, part_o, part_ml, sink=None, softcap=0.0, value_dim=None, gate_channels=False):
     B = q.shape[0]
     _check(lib().cm_attn_decode(dtype_code(q.dtype), _ptr(ctx), ctx.stride(0), _ptr(q), q.stride(0), _ptr(gate),
                                 0 if gate is None else gate.stride(0), _ptr(seq_pos), _ptr(seq_slot), _ptr(pool),
                                 pages, _ptr(ptab), ptab.stride(0), ring, window, B, QH, KVH, HD, n_chunks, scale, softcap,
-                                _ptr(part_o), _ptr(part_ml), _ptr(sink), _stream()), "attn_decode", 2,
+                                _ptr(part_o), _ptr(part_ml), _ptr(sink), value_dim or HD, int(gate_channels), _stream()), "attn_decode", 2,
            cost=lambda: (f"{B} sequences, {QH}/{KVH} heads of {HD}, window {window}, {n_chunks} chunks", 0, 0))
 
 
@@ -787,12 +847,17 @@ def norm_f32in(out, x, w, eps, dyt=None, layer=False):
            cost=lambda: (f"{rows}x{H}", _nbytes(x, out, w), 4 * rows * H))
 
 
+def act_inplace(x, kind):
+    """x <- act(x), in x's dtype (contiguous): kind "relu2" max(x, 0)^2, "gelu_tanh" the tanh form of gelu."""
+    if not x.is_contiguous():
+        raise KernelError("act_inplace takes a contiguous tensor")
+    _check(lib().cm_act_inplace(dtype_code(x.dtype), _ptr(x), x.numel(), {"relu2": 0, "gelu_tanh": 1}[kind], _stream()), kind + "_inplace",
+           cost=lambda: (f"{tuple(x.shape)}", 2 * _nbytes(x), 0))
+
+
 def relu2_inplace(x):
     """x <- max(x, 0)^2, in x's dtype (contiguous)."""
-    if not x.is_contiguous():
-        raise KernelError("relu2_inplace takes a contiguous tensor")
-    _check(lib().cm_relu2_inplace(dtype_code(x.dtype), _ptr(x), x.numel(), _stream()), "relu2_inplace",
-           cost=lambda: (f"{tuple(x.shape)}", 2 * _nbytes(x), 0))
+    act_inplace(x, "relu2")
 
 
 def _term_arrays(terms, rows, H, act, name):
@@ -801,6 +866,10 @@ def _term_arrays(terms, rows, H, act, name):
         raise KernelError(f"{name}: at most four terms")
     terms = [tuple(t) + (None,) * (5 - len(t)) for t in terms]
     for t, _, per_row, index, weights in terms:
+        if per_row == 0:                       # one row for all rows
+            if t.numel() != H or index is not None or weights is not None or not t.is_contiguous() or t.dtype not in (torch.float32, act):
+                raise KernelError(f"{name}: a bias is one row")
+            continue
         fits = t.numel() == rows * per_row * H if index is None else (index.numel() == rows * per_row and t.shape[-1] == H)
         if not t.is_contiguous() or not fits or t.dtype not in (torch.float32, act):
             raise KernelError(f"{name}: a term's shape or dtype does not fit")
@@ -855,6 +924,25 @@ def postnorm_residual(h, terms, h_scale, w, eps, n_out=None, history=None, coef=
                          + sum(rows * t[2] * H * t[0].element_size() for t in terms), (n + 5 + 2 * n_hist) * rows * H))
 
 
+def outnorm_residual(h, terms, w, eps, n_out=None, w_next=None, eps_next=0.0):
+    """The norm on what is added: h (float32, in place) += norm(the sum of `terms`) * w (an RMS norm, w float32 [H]).  n_out
+    (activation dtype, optional) <- h, or with `w_next` norm(h) * w_next: the rows as the next reader takes them."""
+    rows, H = h.shape
+    if h.dtype != torch.float32 or not h.is_contiguous():
+        raise KernelError("outnorm_residual: a contiguous float32 stream")
+    act = n_out.dtype if n_out is not None else next((t[0].dtype for t in terms if t[0].dtype != torch.float32), torch.float32)
+    terms, n, ptrs, scales, per, f32, index, weights = _term_arrays(terms, rows, H, act, "outnorm_residual")
+    for t in (w, w_next):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != H or not t.is_contiguous()):
+            raise KernelError("outnorm_residual: float32 norm weights, one per column")
+    if n_out is not None and (n_out.shape != h.shape or not n_out.is_contiguous()):
+        raise KernelError("outnorm_residual: the rows for the next reader are of the stream's shape")
+    _check(lib().cm_outnorm_residual(dtype_code(act), _ptr(h), _ptr(n_out), n, ptrs, scales, per, f32, index, weights, _ptr(w),
+                                     _ptr(w_next), rows, H, eps, eps_next, _stream()), "outnorm_residual",
+           cost=lambda: (f"{rows}x{H}, {n} terms", 2 * _nbytes(h) + _nbytes(n_out) + sum(rows * t[2] * H * t[0].element_size() for t in terms),
+                         (n + 10) * rows * H))
+
+
 HYPER_MAX_STREAMS = 8              # csrc/hyper.cu: HC_MAX_STREAMS
 
 
@@ -877,6 +965,8 @@ def hyper_connect(x, terms=(), mix=None, put=None, n_out=None, read=None, w=None
     if n_out is not None and (tuple(n_out.shape) != (rows, W) or not n_out.is_contiguous()):
         raise KernelError("hyper_connect: the normed rows are [rows, W]")
     act = n_out.dtype if n_out is not None else next((t[0].dtype for t in terms if t[0].dtype != torch.float32), torch.float32)
+    if any(t[2] == 0 for t in terms):
+        raise KernelError("hyper_connect: a term has pieces for every row")
     terms, n, ptrs, scales, per, f32, index, weights = _term_arrays(terms, rows, W, act, "hyper_connect")
     write = streams if open_ or mix is not None else None
     _check(lib().cm_hyper_connect(dtype_code(act), _ptr(write), _ptr(x), int(open_), _ptr(mix), _ptr(put), _ptr(read), _ptr(w), eps,
@@ -1222,7 +1312,8 @@ class _LatentArgs(ctypes.Structure):
                 ("eps", _f), ("scale", _f), ("rows", _ll), ("tok_pos", _vp), ("tok_seq", _vp), ("seq_start", _vp),
                 ("seq_pos0", _vp), ("seq_end", _vp), ("seq_slot", _vp), ("pool", _vp), ("ptab", _vp), ("ptab_stride", _ll),
                 ("B", _i), ("max_len", _i), ("splits", _i), ("chunk", _i), ("parts", _vp), ("ckv", _vp), ("kvu", _vp),
-                ("ld_kvu", _ll), ("qkv", _vp), ("ld_qkv", _ll), ("HD", _i), ("DV", _i), ("mag", _f), ("no_entry", _i)]
+                ("ld_kvu", _ll), ("qkv", _vp), ("ld_qkv", _ll), ("HD", _i), ("DV", _i), ("mag", _f), ("no_entry", _i),
+                ("window", _i), ("ring", _i), ("no_store", _i), ("sink", _vp)]
 
 
 latent_decode_tensor_cores = True   # off: single-token steps of the latent attention stay on the CUDA cores (tests compare)
@@ -1250,23 +1341,33 @@ def _latent_args(batch, pool, ptab, H, D, R, KR, QR, eps=0.0, scale=1.0, mag=1.0
 
 
 def latent_prepare(cq, proj, q_off, kv_off, wq_norm, wkv_norm, rate, pool, ptab, batch, H, D, R, KR, QR, eps, entries=None,
-                   mag=1.0, make_entry=True):
+                   mag=1.0, make_entry=True, ring=0, store=True):
     """Per row of the step: cq = norm(proj[q_off : q_off + QR]) * wq_norm (activation dtype, for the product that
     makes the heads' queries), and the row's cache entry [norm(proj[kv_off : kv_off + KR]) * wkv_norm | the next R
     channels turned by the position (pairs 2i, 2i + 1 by position * rate[i]) | zeros] into pool [pages, PAGE_TOKENS, EC]
     through the page table.  Norms and angles are float32.  `entries` [rows, EC] (contiguous): the same entries once
     more in the order of the step's rows (zeros for rows of padding), for a product over them.  `mag`: the factor on
     sine and cosine (all rotations of the latent attention take it).  `make_entry` False: only cq is made (a layer that
-    reads another layer's entries; kv_off and wkv_norm are then not used)."""
-    a = _latent_args(batch, pool, ptab, H, D, R, KR, QR, eps=eps, mag=mag, no_entry=int(not make_entry), proj=_ptr(proj), ld_proj=proj.stride(0), q_off=q_off,
+    reads another layer's entries; kv_off and wkv_norm are then not used).  QR = 0 (cq None): no query latent.  `ring`: the pages
+    are a ring of that many entries.  `store` False: only `entries` is written (`latent_store` brings it to the cache later)."""
+    a = _latent_args(batch, pool, ptab, H, D, R, KR, QR, eps=eps, mag=mag, no_entry=int(not make_entry), ring=ring, no_store=int(not store), proj=_ptr(proj), ld_proj=proj.stride(0), q_off=q_off,
                      kv_off=kv_off, cq=_ptr(cq), wq_norm=_ptr(wq_norm), wkv_norm=_ptr(wkv_norm), rate=_ptr(rate),
                      ckv=_ptr(entries))
-    if proj.stride(1) != 1 or not cq.is_contiguous() or cq.dtype != proj.dtype or pool.dtype != proj.dtype:
+    if proj.stride(1) != 1 or pool.dtype != proj.dtype or (QR and (not cq.is_contiguous() or cq.dtype != proj.dtype)):
         raise KernelError("latent_prepare: row-major operands of one dtype")
     if entries is not None and (entries.shape != (batch.T, pool.shape[-1]) or not entries.is_contiguous() or entries.dtype != pool.dtype):
         raise KernelError("latent_prepare: the entries' copy is [rows, entry size] in the cache's dtype")
     _check(lib().cm_latent_prepare(dtype_code(proj.dtype), ctypes.byref(a), _stream()), "latent_prepare",
            cost=lambda: (f"{batch.T} rows, {QR} + {KR} + {R}", batch.T * (2 * QR + 2 * (KR + R)) * proj.element_size(), 6 * batch.T * (QR + KR)))
+
+
+def latent_store(entries, pool, ptab, batch, R, KR, ring=0):
+    """The step's entries [rows, EC] (from `latent_prepare`) into the cache pages; a ring keeps a sequence's last `ring`."""
+    a = _latent_args(batch, pool, ptab, 1, 0, R, KR, 0, ckv=_ptr(entries), ring=ring)
+    if entries.shape != (batch.T, pool.shape[-1]) or not entries.is_contiguous() or entries.dtype != pool.dtype:
+        raise KernelError("latent_store: entries [rows, entry size] in the cache's dtype")
+    _check(lib().cm_latent_store(dtype_code(pool.dtype), ctypes.byref(a), _stream()), "latent_store",
+           cost=lambda: (f"{batch.T} rows", 2 * _nbytes(entries), 0))
 
 
 def latent_query_turn(qa, q, rate, pool, ptab, batch, H, D, R, KR, mag=1.0):
@@ -1312,23 +1413,32 @@ def latent_attn_splits(rows, H, keys, sm_count=148, heads_per_block=32, kv_rank=
     return -(-keys // chunk) if splits > 1 else 1, chunk
 
 
-def latent_attn(out, qa, gate, pool, ptab, batch, H, R, KR, scale, splits=1, chunk=0, parts=None, tensor_cores=False):
+def latent_attn(out, qa, gate, pool, ptab, batch, H, R, KR, scale, splits=1, chunk=0, parts=None, tensor_cores=False, window=0,
+                ring=0, sink=None, entries=None):
     """Causal softmax attention of every head's query row qa [rows, H, KR + R] (float32) over the cache entries of
     its sequence (positions <= the row's own); out [rows, H, KR] (float32) = the weights' sum over the latents,
     times sigmoid(gate[t, h]) when `gate` ([rows, >= H] logits, activation dtype) is given.  `splits` > 1: the keys
     are cut into runs of `chunk` entries, each run a block of its own, merged afterwards (`parts`: float32 scratch of
     rows * H * splits * (2 + KR)).  `tensor_cores`: a step of one token per sequence over a bfloat16 cache takes the
-    mma.sync form (the queries rounded to bfloat16, sums in float32)."""
+    mma.sync form (the queries rounded to bfloat16, sums in float32).  `window` W > 0: a row sees the last W positions (runs of
+    keys are then counted from the tile of the first one); `ring`: the pages are a ring of that many entries; `sink` (float32
+    [H]): a logit per head in the softmax's denominator, without key and value; `entries` [rows, EC]: positions of the step are
+    read from there instead of the cache (CUDA-core form)."""
     a = _latent_args(batch, pool, ptab, H, 0, R, KR, 0, scale=scale, qa=_ptr(qa), ldqa=qa.stride(0), gate=_ptr(gate),
-                     ld_gate=0 if gate is None else gate.stride(0), out=_ptr(out), ldo=out.stride(0))
+                     ld_gate=0 if gate is None else gate.stride(0), out=_ptr(out), ldo=out.stride(0), window=window, ring=ring,
+                     sink=_ptr(sink), ckv=_ptr(entries))
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != H):
+        raise KernelError("latent_attn: a float32 sink per head")
+    if entries is not None and (entries.shape != (batch.T, pool.shape[-1]) or not entries.is_contiguous() or entries.dtype != pool.dtype):
+        raise KernelError("latent_attn: the step's entries are [rows, entry size] in the cache's dtype")
     a.splits, a.chunk, a.parts = splits, chunk, _ptr(parts)
     if qa.dtype != torch.float32 or out.dtype != torch.float32 or (gate is not None and gate.dtype != pool.dtype):
         raise KernelError("latent_attn: float32 queries and sums")
     if splits > 1 and (parts is None or parts.numel() < batch.T * H * splits * (2 + KR)):
         raise KernelError("latent_attn: the splits' scratch is missing or short")
     cost = lambda: (f"{batch.B} sequences, {batch.T} rows, {H} heads over {KR}+{R}",
-                    _nbytes(qa, out) + sum((p + n) * pool.shape[-1] * pool.element_size() for p, n in zip(batch.positions, batch.lengths)),
-                    sum(2 * n * H * (p + (n + 1) // 2) * (2 * KR + R) for p, n in zip(batch.positions, batch.lengths)))
+                    _nbytes(qa, out) + sum((min(p + n, window + n) if window else p + n) * pool.shape[-1] * pool.element_size() for p, n in zip(batch.positions, batch.lengths)),
+                    sum(2 * n * H * (min(p + (n + 1) // 2, window) if window else p + (n + 1) // 2) * (2 * KR + R) for p, n in zip(batch.positions, batch.lengths)))
     if tensor_cores:
         if batch.kind != "decode" or batch.T != batch.B or pool.dtype != torch.bfloat16:
             raise KernelError("latent_attn: the tensor-core form takes one token per sequence over a bfloat16 cache")
@@ -1337,19 +1447,23 @@ def latent_attn(out, qa, gate, pool, ptab, batch, H, R, KR, scale, splits=1, chu
     _check(lib().cm_latent_attn(dtype_code(pool.dtype), ctypes.byref(a), _stream()), "latent_attn", 2 if splits > 1 else 1, cost=cost)
 
 
-def head_linear(y, x, w, H, x_size, y_size):
+def head_linear(y, x, w, H, x_size, y_size, gate=None):
     """A matrix per head: y[t, h * y_size + n] = sum_k x[t, h * x_size + k] * w[h, n, k] for w [H, N, K].  x and y are
-    in w's dtype or float32 (a sum that stays unrounded between two steps)."""
+    in w's dtype or float32 (a sum that stays unrounded between two steps).  `gate` [rows, >= H N] (w's dtype): a logit per
+    result, whose sigmoid multiplies it before the rounding."""
     rows = x.shape[0]
     N, K = w.shape[1], w.shape[2]
     if x.stride(1) != 1 or y.stride(1) != 1 or not w.is_contiguous() or w.shape[0] != H:
         raise KernelError("head_linear: row-major operands, one matrix per head")
+    if gate is not None and (gate.dtype != w.dtype or gate.stride(1) != 1 or gate.shape[0] != rows or gate.shape[1] < H * N):
+        raise KernelError("head_linear: gate logits [rows, >= heads x columns] in the matrices' dtype")
     for t in (x, y):
         if t.dtype not in (w.dtype, torch.float32):
             raise KernelError("head_linear: rows in the matrices' dtype or float32")
     _check(lib().cm_head_linear(dtype_code(w.dtype), _ptr(y), _ptr(x), _ptr(w), rows, H, N, K, x.stride(0), y.stride(0), x_size,
                                 y_size, int(x.dtype == torch.float32 and w.dtype != torch.float32),
-                                int(y.dtype == torch.float32 and w.dtype != torch.float32), _stream()), "head_linear",
+                                int(y.dtype == torch.float32 and w.dtype != torch.float32), _ptr(gate),
+                                0 if gate is None else gate.stride(0), _stream()), "head_linear",
            cost=lambda: (f"{rows} rows, {H} heads of {N}x{K}", rows * H * (N * y.element_size() + K * x.element_size()) + _nbytes(w),
                          2 * rows * H * N * K))
 

@@ -1,2 +1,2 @@
 """Architectures.  Importing this package registers them by name."""
-from . import fozedra, kofadra, lfm3, maferax, narasun, relilix  # noqa: F401
+from . import fozedra, kofadra, lfm3, maferax, mogilorn, narasun, relilix  # noqa: F401

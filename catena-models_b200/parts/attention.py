@@ -35,6 +35,13 @@ start, before the rotation (K = 1 is a factor per channel; 0: no filter and no t
 rows of a sequence are part of the layer's state (float32, a ring beside the key/value pages).  `value_from_key`: the layer has no value projection; a position's value is its key
 as the filter leaves it, before the rotation.  Filter, rotation and the cache write are one kernel
 (`kernels.tap_rotate_store`), which leaves the step's rows as [q | turned k | v] for the attention kernels.
+
+`bias`: q, k, v and the output projection have biases (`q_bias`, `k_bias`, `v_bias`, `out_bias` name the tensors).
+`gate_channels` (with `output_gate`): the gate has a logit per channel of the concatenated heads instead of one per head.
+`value_mix` = (role, name): values are mixed with those of another layer of the same step, v <- (1 - a) v + a v_first, before
+they are cached; `name` is the tensor of the one number a, role "source" marks the layer whose own values (with their bias) are
+v_first (its number is not used), "mix" the layers that mix.  With a bias, a mix or a position encoding that turns part of a
+head (`position.dims`), everything between the projection and the attention is one kernel (`kernels.head_prepare`).
 """
 from __future__ import annotations
 
@@ -56,11 +63,23 @@ class GQAttention(Mixer):
 
     def __init__(self, prefix, hidden, heads, kv_heads, head_dim, window, position, qk_norm_eps,
                  output_gate, names=None, shares_kv=False, scale=None, sink_name=None, q_temp=None, value_dim=None,
-                 out_dtype=None, softcap=0.0, taps=0, value_from_key=False, chunk=0, sink_value=None):
+                 out_dtype=None, softcap=0.0, taps=0, value_from_key=False, chunk=0, sink_value=None, bias=False,
+                 gate_channels=False, value_mix=None):
         names = names or {}
         n = lambda key, default: prefix + names.get(key, default)
         qk_dim, v_dim = head_dim, value_dim or head_dim
-        if v_dim != qk_dim or (scale is not None and qk_dim % 16):
+        self.bias, self.value_mix = bool(bias), value_mix
+        self.gate_channels = bool(gate_channels) and bool(output_gate)
+        filtered = bool(taps) or bool(value_from_key)
+        self.one_prepare = not filtered and (self.bias or value_mix is not None or bool(getattr(position, "dims", 0)))
+        if value_mix is not None and value_mix[0] not in ("source", "mix"):
+            raise ValueError("GQAttention: value_mix ('source' | 'mix', tensor name)")
+        if (self.one_prepare or self.gate_channels) and (shares_kv or q_temp or filtered):
+            raise ValueError("GQAttention: biases, mixed values, partial rotation and gates per channel go with neither shared keys, "
+                             "filters nor a query temperature")
+        if self.bias and out_dtype != "float32":
+            raise ValueError("GQAttention: the output bias joins a float32 residual sum")
+        if v_dim != qk_dim or ((scale is not None or self.one_prepare) and qk_dim % 16):
             head_dim = -(-max(qk_dim, v_dim) // 16) * 16       # one padded head size for q, k and v
         pad_qk = (heads, qk_dim, head_dim) if head_dim != qk_dim else None
         pad_k = (kv_heads, qk_dim, head_dim) if head_dim != qk_dim else None
@@ -74,7 +93,7 @@ class GQAttention(Mixer):
         if (self.taps > 0 or self.value_from_key) and (shares_kv or qk_norm_eps is not None or q_temp or output_gate):
             raise ValueError("GQAttention: the filtered form has neither head norm, query temperature, gate nor shared keys")
         self.filtered = self.taps > 0 or self.value_from_key
-        if self.filtered:
+        if self.filtered or self.one_prepare:
             self.fused_decode_ok = False       # its decode step runs a kernel of its own between the products
         self.sink_name, self.sink = (prefix + sink_name if sink_name else None), None
         self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp else None
@@ -106,11 +125,16 @@ class GQAttention(Mixer):
                 pads.append(pad_v)
         if self.output_gate:
             mats.append(n("gate", "attn_gate.weight"))
-            rows.append(heads)
+            rows.append(heads * v_dim if self.gate_channels else heads)
             pads.append(None)
-        self.qkvg = Linear(mats, rows, hidden, head_rows=pads)
+        self.qkvg = Linear(mats, rows, hidden, head_rows=pads, row_multiple=8 if self.one_prepare or self.gate_channels else 1)
+        # channels of a head that the attention leaves: all, or with a gate per channel those that are no padding
+        self.ctx_dim = v_dim if self.gate_channels else head_dim
+        self.bias_names = [n("q_bias", "attn_q.bias"), n("k_bias", "attn_k.bias"), n("v_bias", "attn_v.bias")] if self.bias else []
+        self.out_bias_name = n("out_bias", "attn_output.bias") if self.bias else None
+        self.qkv_bias = self.out_bias = self.mix_share = None
         self.out = Linear(n("out", "attn_output.weight"), hidden, heads * v_dim,
-                          head_cols=(heads, v_dim, head_dim) if head_dim != v_dim else None)
+                          head_cols=(heads, v_dim, head_dim) if head_dim != v_dim and not self.gate_channels else None)
         self.q_norm_name, self.k_norm_name = n("q_norm", "attn_q_norm.weight"), n("k_norm", "attn_k_norm.weight")
         self.q_norm_w = self.k_norm_w = None
         self.tap_names = (n("q_taps", "attn_q.conv"), n("k_taps", "attn_k.conv")) if self.taps > 0 else ()
@@ -128,6 +152,11 @@ class GQAttention(Mixer):
         if self.taps > 0:
             specs += [TensorSpec(self.tap_names[0], (self.heads * self.qk_dim, self.taps), "conv"),
                       TensorSpec(self.tap_names[1], (self.kv_heads * self.qk_dim, self.taps), "conv")]
+        if self.bias:
+            sizes = [self.heads * self.qk_dim, self.kv_heads * self.qk_dim, self.kv_heads * self.v_dim, self.hidden]
+            specs += [TensorSpec(name, (size,), "vector") for name, size in zip(self.bias_names + [self.out_bias_name], sizes)]
+        if self.value_mix is not None:
+            specs.append(TensorSpec(self.value_mix[1], (), "vector"))
         if self.qk_norm_eps is None:
             return specs
         specs.append(TensorSpec(self.q_norm_name, (self.qk_dim,), "norm"))
@@ -150,6 +179,16 @@ class GQAttention(Mixer):
             else:
                 self.tap_w = torch.ones((self.q_size + self.kv_size, 1), dtype=torch.float32, device=rt.device)
             self._bound.append(self.tap_w)
+        if self.bias:
+            parts = []
+            for name, size in zip(self.bias_names, (self.qk_dim, self.qk_dim, self.v_dim)):
+                parts.append(torch.nn.functional.pad(tensors[name].to(torch.float32).view(-1, size), (0, self.head_dim - size)).reshape(-1))
+            self.qkv_bias = torch.cat(parts).contiguous()
+            self.out_bias = tensors[self.out_bias_name].to(torch.float32).contiguous()
+            self._bound += [self.qkv_bias, self.out_bias]
+        if self.value_mix is not None and self.value_mix[0] == "mix":
+            self.mix_share = tensors[self.value_mix[1]].to(torch.float32).reshape(1).contiguous()
+            self._bound.append(self.mix_share)
         if self.sink_name:
             self.sink = tensors[self.sink_name].to(torch.float32).contiguous()
             self._bound.append(self.sink)
@@ -207,6 +246,22 @@ class GQAttention(Mixer):
                                      softcap=self.softcap)
         return self.out.apply(rt, ctx, out_dtype=self.out_dtype)
 
+    def _prepare(self, batch, proj, state):
+        """Biases, head norms, rotation, mixed values and (except in an append step) the cache write, in place."""
+        QS, KVS, HD = self.q_size, self.kv_size, self.head_dim
+        mix = None
+        if self.mix_share is not None:
+            if "v_first" not in batch.shared:
+                raise ValueError("GQAttention: mixed values need an earlier layer of the step with value_mix ('source', ...)")
+            mix = (*batch.shared["v_first"], self.mix_share)
+        kv = None if batch.append else (state.pool, state.pages, state.ptab, state.ring)
+        kernels.head_prepare(proj, batch, self.heads, self.kv_heads, HD, bias=self.qkv_bias, wq=self.q_norm_w, wk=self.k_norm_w,
+                             norm_dim=self.qk_dim, eps=self.qk_norm_eps or 0.0, rate=self.position.rate_table(),
+                             interleaved=self.position.pairing == "interleaved", mag=getattr(self.position, "magnitude", 1.0),
+                             value_dim=self.v_dim, mix=mix, kv=kv)
+        if self.value_mix is not None and self.value_mix[0] == "source":
+            batch.shared["v_first"] = (proj[:, QS + KVS:QS + 2 * KVS], self.v_dim, HD)
+
     def forward(self, rt, batch, x, state):
         QS, KVS, QH, KVH, HD = self.q_size, self.kv_size, self.heads, self.kv_heads, self.head_dim
         if self.filtered:
@@ -216,7 +271,10 @@ class GQAttention(Mixer):
                              "by the plan (owns_state=False), and only such a layer")
         proj = self.qkvg.apply(rt, x)                  # [T, QS + 2 KVS (+ QH)], or [T, QS (+ QH)] when sharing
         interleaved = self.position.pairing == "interleaved"
-        if self.shares_kv:
+        if self.one_prepare:
+            self._prepare(batch, proj, state)
+            gate = proj[:, QS + 2 * KVS:] if self.output_gate else None
+        elif self.shares_kv:
             # q only: head norm and rotation over the q heads, nothing written to the cache
             kernels.qk_prepare(proj, self.q_norm_w, None, self.position.rate_table(), batch.tok_pos, batch.tok_seq,
                                batch.seq_slot, batch.seq_end, None, 0, None, 0, QH, 0, HD, self.qk_norm_eps or 0.0,
@@ -231,7 +289,8 @@ class GQAttention(Mixer):
                                norm_dim=self.qk_dim)
             gate = proj[:, QS + 2 * KVS:] if self.output_gate else None
         q = proj[:, :QS]
-        ctx = torch.empty((batch.T, QS), dtype=x.dtype, device=x.device)
+        ctx = torch.empty((batch.T, QH * self.ctx_dim), dtype=x.dtype, device=x.device)
+        stored = {"value_dim": self.ctx_dim, "gate_channels": self.gate_channels}
         if batch.prefill or batch.append:
             if self.shares_kv and batch.append and state.ring:
                 raise NotImplementedError("an append step of a layer that shares the keys and values of a sliding "
@@ -250,13 +309,13 @@ class GQAttention(Mixer):
                 batch.shared[("kv", state.unit)] = (k, v)
             if batch.append:
                 rt.attention_append(ctx, q, k, v, gate, batch, state, QH, KVH, HD, self.mask, self.scale, sink=self.sink,
-                                    softcap=self.softcap)
+                                    softcap=self.softcap, **stored)
                 if not self.shares_kv:
                     kernels.kv_store(proj[:, QS:QS + 2 * KVS], batch.tok_pos, batch.tok_seq, batch.seq_slot,
                                      batch.seq_end, state.pool, state.pages, state.ptab, state.ring, KVH, HD)
             else:
                 rt.attention_prefill(ctx, q, k, v, gate, batch, QH, KVH, HD, self.mask, self.scale, sink=self.sink,
-                                     softcap=self.softcap)
+                                     softcap=self.softcap, **stored)
         else:
             # launched for the longest sequence that this step's length class allows, so that a
             # recording of the step serves every step of the class
@@ -265,7 +324,9 @@ class GQAttention(Mixer):
             part_o, part_ml = rt.scratch_attn_decode(batch.B, QH, HD, n_chunks)
             kernels.attn_decode(ctx, q, gate, batch.seq_pos0, batch.seq_slot, state.pool, state.pages, state.ptab,
                                 state.ring, self.mask, QH, KVH, HD, n_chunks, self.scale, part_o, part_ml, sink=self.sink,
-                                softcap=self.softcap)
+                                softcap=self.softcap, **stored)
+        if self.bias:
+            return kernels.Terms([(self.out.apply(rt, ctx, out_dtype=self.out_dtype), 1.0, 1), (self.out_bias, 1.0, 0)])
         return self.out.apply(rt, ctx, out_dtype=self.out_dtype, partial_ok=batch.partial_sums_ok and self.out_dtype is None)
 
 

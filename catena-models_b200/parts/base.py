@@ -156,6 +156,7 @@ class Position(Part):
 
 class Block(Part):
     input_norm = None
+    reads_stream = False     # True: a block without an input norm that takes the stream in the activation dtype as `n`
 
     def state_spec(self):
         return None

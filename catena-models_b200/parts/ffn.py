@@ -70,6 +70,29 @@ class ReluSquared(FeedForward):
         return self.down.apply(rt, a, out_dtype=self.out_dtype, partial_ok=batch.partial_sums_ok and self.out_dtype is None)
 
 
+class GeluTanh(FeedForward):
+    """Plain two-matrix feed-forward with the tanh form of gelu between: W_down gelu(W_up x), the activation in the epilogue of
+    the first product."""
+    prompt_capturable = True
+    supports_append = True
+
+    def __init__(self, prefix, hidden, intermediate, names=None, out_dtype=None):
+        import torch
+
+        self.out_dtype = {None: None, "float32": torch.float32}[out_dtype]
+        names = names or {}
+        self.hidden, self.intermediate = hidden, intermediate
+        self.up = Linear(prefix + names.get("up", "up"), intermediate, hidden)
+        self.down = Linear(prefix + names.get("down", "down"), hidden, intermediate)
+
+    def children(self):
+        return [self.up, self.down]
+
+    def forward(self, rt, batch, x):
+        a = rt.linear_gelu(x, self.up.weight)
+        return self.down.apply(rt, a, out_dtype=self.out_dtype, partial_ok=batch.partial_sums_ok and self.out_dtype is None)
+
+
 class SumOfFeedForwards(FeedForward):
     """Several feed-forwards that read the same input; the result is the sum of theirs (a routed feed-forward and an
     expert that every token runs, say).  Each member hands over a tensor or `kernels.Terms`; the block's residual sum
@@ -96,5 +119,6 @@ class SumOfFeedForwards(FeedForward):
 
 
 register_part("feed_forward", "swiglu", SwiGLU)
+register_part("feed_forward", "gelu_tanh", GeluTanh)
 register_part("feed_forward", "sum", SumOfFeedForwards)
 register_part("feed_forward", "relu_squared", ReluSquared)

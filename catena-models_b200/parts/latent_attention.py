@@ -22,12 +22,18 @@ The position encoding turns the leading `position.dims` channels of the rot_dim 
 channels of that part pass unchanged.  A position encoding with a `magnitude` has it on every sine and cosine, of the
 queries' turned part and of the cached key part alike.
 
+`q_rank` None: the queries come straight from the input, q = W_q h (no query latent).  `gate_channels` (with `output_gate`):
+W_g has a row per channel of the concatenated heads.  `sink_name`: a learned logit per head that joins the softmax's
+denominator and has neither key nor value.  `window` W: position i sees the last W positions, itself among them.  A layer with a
+window keeps a ring of that many entries per sequence; a step of more than one token a sequence then reads its own positions
+from the step's entries, kept side by side, and older ones from the ring, and writes the ring afterwards.
+
 `shares_latents`: the layer has no W_dkv.  It reads the entries [c | r] that another layer of the same latent size and
 rotation wrote (the plan hands it that layer's state unit, `owns_state=False`), with its own W_uk, W_uv, queries and
 gate; in a whole-prompt step of the expanded form it takes the owner's side-by-side copy of the step's entries from
 `StepBatch.shared`.
 
-Every kind of step writes its entries to the cache first.  Portions, single tokens and mixed lengths then read all
+Without a window every kind of step writes its entries to the cache first.  Portions, single tokens and mixed lengths then read all
 keys from there (`kernels.latent_attn`, CUDA cores, float32 sums).  A bfloat16 step of whole prompts has a second form:
 the step's entries, kept side by side, are multiplied by [W_uk; W_uv] into keys and values per head (the turned part
 copied behind each head's key), heads padded with zeros to the 64 or 128 channels of the tensor-core attention kernels
@@ -50,52 +56,74 @@ class LatentAttention(Mixer):
     supports_append = True
 
     def __init__(self, prefix, hidden, heads, dim, rot_dim, value_dim, kv_rank, q_rank, position, scale, eps,
-                 output_gate=True, out_dtype=None, shares_latents=False):
-        if min(heads, dim, value_dim, kv_rank, q_rank) < 1 or rot_dim < 0:
+                 output_gate=True, out_dtype=None, shares_latents=False, window=0, sink_name=None, gate_channels=False):
+        if min(heads, dim, value_dim, kv_rank, 1 if q_rank is None else q_rank) < 1 or rot_dim < 0 or window < 0:
             raise ValueError("LatentAttention: sizes must be positive")
         if getattr(position, "dims", 0) and position.pairing != "interleaved":
             raise ValueError("LatentAttention: the turned part is paired 2i with 2i + 1")
         self.prefix, self.hidden = prefix, hidden
         self.heads, self.dim, self.rot_dim, self.value_dim = heads, dim, rot_dim, value_dim
-        self.kv_rank, self.q_rank = kv_rank, q_rank
+        self.kv_rank, self.q_rank = kv_rank, q_rank or 0
+        self.window, self.sink_name, self.sink = int(window or 0), prefix + sink_name if sink_name else None, None
+        self.gate_channels = bool(gate_channels) and bool(output_gate)
+        if shares_latents and (self.window or q_rank is None):
+            raise ValueError("LatentAttention: shared latents go with neither a window nor queries straight from the input")
         self.position, self.scale, self.eps = position, float(scale), float(eps)
         self.output_gate = bool(output_gate)
         self.shares_latents = bool(shares_latents)
         self.magnitude = float(getattr(position, "magnitude", 1.0))
         self.out_dtype = {None: None, "float32": torch.float32}[out_dtype]
         self.entry = kernels.latent_entry_size(kv_rank, rot_dim)
+        if q_rank is None:
+            # q | gate | latent rows: the gate's columns begin where the queries' do, aligned for the attention kernels
+            H, q_rows = heads, heads * (dim + rot_dim)
+            gate_rows = (H * value_dim if self.gate_channels else H) if self.output_gate else 0
+            self.gate_off, self.kv_off = q_rows, q_rows + gate_rows
+            self.down = Linear([prefix + "q"] + ([prefix + "g"] if gate_rows else []) + [prefix + "dkv"],
+                               [q_rows] + ([gate_rows] if gate_rows else []) + [kv_rank + rot_dim], hidden, row_multiple=8)
+            self.up_q = None
+        else:
+            self._low_rank_queries(prefix, hidden, q_rank)
+        self.out = Linear(prefix + "o", hidden, heads * value_dim)
+        self.wq_norm = self.wkv_norm = self.w_uk_t = self.w_uv = self.w_kvu = self.rate = None
+        # the padded head of the expanded prompt form (0: heads too large for the tensor-core attention kernels)
+        need = max(dim + rot_dim, value_dim)
+        self.expand_head = 64 if need <= 64 else (128 if need <= 128 else 0)
+        # prompts from this many tokens on take the expanded form; shorter ones give its products too few rows
+        self.expand_min_tokens = 64
+
+    def _low_rank_queries(self, prefix, hidden, q_rank):
+        heads, dim, rot_dim, kv_rank = self.heads, self.dim, self.rot_dim, self.kv_rank
         names, rows = [prefix + "dq"], [q_rank]
+        self.kv_off = q_rank
         if not self.shares_latents:
             names.append(prefix + "dkv")
             rows.append(kv_rank + rot_dim)
         self.gate_off = sum(rows)                       # where the gate logits begin in the packed product's rows
         if self.output_gate:
             names.append(prefix + "g")
-            rows.append(heads)
+            rows.append(heads * self.value_dim if self.gate_channels else heads)
         self.down = Linear(names, rows, hidden)
         self.up_q = Linear(prefix + "uq", heads * (dim + rot_dim), q_rank)
-        self.out = Linear(prefix + "o", hidden, heads * value_dim)
-        self.wq_norm = self.wkv_norm = self.w_uk_t = self.w_uv = self.w_kvu = self.rate = None
-        # the padded head of the expanded prompt form (0: heads too large for the tensor-core attention kernels)
-        need = max(dim + rot_dim, value_dim)
-        self.expand_head = 64 if need <= 64 else (128 if need <= 128 else 0)
-        # Prompts from this many tokens on take the expanded form.  Measured on B200, one prompt, 16 heads of 64 + 32 and
-        # 64 over latents of 256, CUDA-core form against expanded form: EXPAND_TABLE
-        self.expand_min_tokens = 64
 
     def children(self):
-        return [self.down, self.up_q, self.out, self.position]
+        return [p for p in (self.down, self.up_q, self.out, self.position) if p is not None]
 
     def tensor_specs(self):
         p = self.prefix
         own = [] if self.shares_latents else [TensorSpec(p + "dkv.norm", (self.kv_rank,), "norm")]
-        return [TensorSpec(p + "dq.norm", (self.q_rank,), "norm")] + own + [
+        if self.q_rank:
+            own = [TensorSpec(p + "dq.norm", (self.q_rank,), "norm")] + own
+        if self.sink_name:
+            own.append(TensorSpec(self.sink_name, (self.heads,), "vector"))
+        return own + [
                 TensorSpec(p + "uk", (self.heads * self.dim, self.kv_rank)),
                 TensorSpec(p + "uv", (self.heads * self.value_dim, self.kv_rank))]
 
     def bind(self, tensors, rt):
         p, H = self.prefix, self.heads
-        self.wq_norm = tensors[p + "dq.norm"].to(torch.float32).contiguous()
+        self.wq_norm = tensors[p + "dq.norm"].to(torch.float32).contiguous() if self.q_rank else None
+        self.sink = tensors[self.sink_name].to(torch.float32).contiguous() if self.sink_name else None
         self.wkv_norm = None if self.shares_latents else tensors[p + "dkv.norm"].to(torch.float32).contiguous()
         # W_uk^T per head [H, kv_rank, dim]: the query side's product; W_uv per head [H, value_dim, kv_rank]
         self.w_uk_t = tensors[p + "uk"].view(H, self.dim, self.kv_rank).transpose(1, 2).contiguous()
@@ -109,10 +137,10 @@ class LatentAttention(Mixer):
         self.rate = rate
         # [W_uk; W_uv] as stored, [H dim + H value_dim, kv_rank]: the expanded prompt form's product
         self.w_kvu = torch.cat([tensors[p + "uk"], tensors[p + "uv"]], 0).contiguous()
-        self._bound = [t for t in (self.wq_norm, self.wkv_norm, self.w_uk_t, self.w_uv, self.w_kvu) if t is not None]
+        self._bound = [t for t in (self.wq_norm, self.wkv_norm, self.w_uk_t, self.w_uv, self.w_kvu, self.sink) if t is not None]
 
     def state_spec(self):
-        return None if self.shares_latents else KVStateSpec(1, self.entry, 0, planes=1)
+        return None if self.shares_latents else KVStateSpec(1, self.entry, self.window, planes=1)
 
     def forward(self, rt, batch, x, state):
         H, D, R, DV, KR, QR = self.heads, self.dim, self.rot_dim, self.value_dim, self.kv_rank, self.q_rank
@@ -125,35 +153,34 @@ class LatentAttention(Mixer):
             raise ValueError("the state unit's entries are not of this layer's latent size")
         pool, ptab = state.pool, state.ptab
         G0, mag = self.gate_off, self.magnitude
-        proj = self.down.apply(rt, x)                                   # [T, QR (+ KR + R) (+ H)]
-        cq = torch.empty((T, QR), dtype=x.dtype, device=dev)
+        ring = state.spec.ring
+        proj = self.down.apply(rt, x)                                   # [T, QR (+ KR + R) (+ gate)], or [T, H (D + R) (+ gate) + KR + R]
+        gate = proj[:, G0:] if self.output_gate else None
+        head_gate, channel_gate = (None, gate) if self.gate_channels else (gate, None)
         HD = self.expand_head
         expand = (batch.kind == "prefill" and HD > 0 and x.dtype == torch.bfloat16 and rt.tensor_core_prompts
                   and batch.max_len >= self.expand_min_tokens and KR % 8 == 0)
+        # a step that reads its own positions from its entries: a ring does not hold them all
+        beside = ring > 0 and batch.kind != "decode"
         if expand and self.shares_latents:
             entries = batch.shared.get(("latent_entries", unit))
             expand = entries is not None
         else:
-            entries = torch.empty((T, self.entry), dtype=x.dtype, device=dev) if expand else None
+            entries = torch.empty((T, self.entry), dtype=x.dtype, device=dev) if expand or beside else None
             if expand:
                 batch.shared[("latent_entries", unit)] = entries      # for the layers that read this one's latents
-        kernels.latent_prepare(cq, proj, 0, QR, self.wq_norm, self.wkv_norm, self.rate, pool, ptab, batch, H, D, R, KR, QR,
+        cq = torch.empty((T, QR), dtype=x.dtype, device=dev) if QR else None
+        kernels.latent_prepare(cq, proj, 0, self.kv_off, self.wq_norm, self.wkv_norm, self.rate, pool, ptab, batch, H, D, R, KR, QR,
                                self.eps, entries=None if self.shares_latents else entries, mag=mag,
-                               make_entry=not self.shares_latents)
-        q = self.up_q.apply(rt, cq)                                      # [T, H (D + R)]
+                               make_entry=not self.shares_latents, ring=ring, store=not (beside and batch.append))
+        q = self.up_q.apply(rt, cq) if QR else proj[:, :H * (D + R)]     # [T, H (D + R)]
         if expand:
             kvu = rt.linear(entries[:, :KR], self.w_kvu)                 # [T, H D + H DV]
             qkv = torch.empty((T, 3 * H * HD), dtype=x.dtype, device=dev)
             kernels.latent_expand(qkv, q, kvu, entries, self.rate, pool, ptab, batch, H, D, R, DV, KR, HD, mag=mag)
-            wide = torch.empty((T, H * HD), dtype=x.dtype, device=dev)
-            rt.attention_prefill(wide, qkv[:, :H * HD], qkv[:, H * HD:2 * H * HD], qkv[:, 2 * H * HD:],
-                                 proj[:, G0:] if self.output_gate else None, batch, H, H, HD, 0, self.scale)
-            if HD == DV:
-                ctx = wide
-            else:
-                ctx = torch.empty((T, H, DV), dtype=x.dtype, device=dev)
-                ctx.copy_(wide.view(T, H, HD)[:, :, :DV])
-                ctx = ctx.view(T, H * DV)
+            ctx = torch.empty((T, H * DV), dtype=x.dtype, device=dev)
+            rt.attention_prefill(ctx, qkv[:, :H * HD], qkv[:, H * HD:2 * H * HD], qkv[:, 2 * H * HD:], gate, batch, H, H, HD,
+                                 self.window, self.scale, sink=self.sink, value_dim=DV, gate_channels=self.gate_channels)
             return self.out.apply(rt, ctx, out_dtype=self.out_dtype)
         qa = torch.empty((T, H * (KR + R)), dtype=torch.float32, device=dev)
         kernels.head_linear(qa, q, self.w_uk_t, H, D + R, KR + R)
@@ -167,13 +194,17 @@ class LatentAttention(Mixer):
         if batch.kind == "decode":
             # sized by the longest sequence that the step's class of lengths allows, so that a recording serves the class
             keys = state.spec.entries(state.spec.length_class(batch.max_end))
+            if self.window:
+                keys = min(keys, self.window) + kernels.LATENT_KEY_TILE      # key tiles begin in front of the window
             splits, chunk = kernels.latent_attn_splits(T, H, keys, heads_per_block=16 if mma else 32, kv_rank=KR)
             if splits > 1:
                 parts = rt.scratch("latent_attn_parts", T * H * splits * (2 + KR))
-        kernels.latent_attn(sums, qa, proj[:, G0:] if self.output_gate else None, pool, ptab, batch, H, R, KR,
-                            self.scale, splits=splits, chunk=chunk, parts=parts, tensor_cores=mma)
+        kernels.latent_attn(sums, qa, head_gate, pool, ptab, batch, H, R, KR, self.scale, splits=splits, chunk=chunk, parts=parts,
+                            tensor_cores=mma, window=self.window, ring=ring, sink=self.sink, entries=entries if beside else None)
         ctx = torch.empty((T, H * DV), dtype=x.dtype, device=dev)
-        kernels.head_linear(ctx, sums, self.w_uv, H, KR, DV)
+        kernels.head_linear(ctx, sums, self.w_uv, H, KR, DV, gate=channel_gate)
+        if beside and batch.append:
+            kernels.latent_store(entries, pool, ptab, batch, R, KR, ring=ring)
         return self.out.apply(rt, ctx, out_dtype=self.out_dtype)
 
 

@@ -18,11 +18,12 @@ class Linear(Part):
     fused_decode_ok = True
     supports_append = True
 
-    def __init__(self, names, rows, in_features, role="matrix", head_rows=None, head_cols=None):
+    def __init__(self, names, rows, in_features, role="matrix", head_rows=None, head_cols=None, row_multiple=1):
         """head_rows: per tensor None or (heads, size, padded size): the tensor's rows are `heads` blocks of
         `size`, and each block is followed by padded - size rows of zeros in the bound matrix (outputs that
         are zero: a kernel with a fixed head size can then run heads of another size).  head_cols: the same
-        for the columns of a single tensor (zero columns meet the padding of its input)."""
+        for the columns of a single tensor (zero columns meet the padding of its input).  row_multiple: rows of zeros fill the
+        bound matrix up to a multiple of this (so that the product's rows begin at aligned addresses)."""
         self.names = [names] if isinstance(names, str) else list(names)
         self.rows = [rows] if isinstance(rows, int) else list(rows)
         self.in_features = in_features
@@ -31,13 +32,16 @@ class Linear(Part):
         self.head_rows = list(head_rows) if head_rows else [None] * len(self.names)
         self.head_cols = head_cols
         self.bound_rows = [r if p is None else p[0] * p[2] for r, p in zip(self.rows, self.head_rows)]
-        self.out_features = sum(self.bound_rows)
+        self.fill_rows = -sum(self.bound_rows) % row_multiple
+        self.out_features = sum(self.bound_rows) + self.fill_rows
 
     def tensor_specs(self):
         return [TensorSpec(n, (r, self.in_features), self.role) for n, r in zip(self.names, self.rows)]
 
     def bind(self, tensors, rt):
         parts = [self._padded(tensors[n], p) for n, p in zip(self.names, self.head_rows)]
+        if self.fill_rows:
+            parts.append(torch.zeros((self.fill_rows, self.in_features), dtype=parts[0].dtype, device=parts[0].device))
         if len(parts) == 1:
             self.weight = parts[0]
         else:

@@ -14,6 +14,8 @@ feed-forward, each sum with a constant factor.
 sublayers read the stream itself.  Optionally followed by an average over the depth of the stack: what the next layer
 reads is a weighted sum of the embedding output and of every layer's result so far.
 
+`OutputNormBlock`: the norm on what a sublayer adds: h <- h + norm1(mixer(h)), then h <- h + norm2(feed_forward(h)).
+
 `HyperBlock`: the sequential arrangement on hyper-connected streams: the residual is several copies per token, a sublayer
 reads their weighted sum and its result is written back to all of them with a mix between them.
 
@@ -209,6 +211,55 @@ class PostNormBlock(Block):
         return h, self._sum(rt, batch, h, f, self.ffn_norm, True, cast_last)
 
 
+class OutputNormBlock(Block):
+    """Two sublayers one after the other on a float32 stream, each with a norm on what it adds and none in front of it:
+    h <- h + norm1(mixer(h)), then h <- h + norm2(feed_forward(h)).  Both sublayers read the stream itself (in the activation
+    dtype); the feed-forward and its norm may be absent together.  The sum of a sublayer's terms, its norm, the residual sum and
+    the rounding (or the norm) of the rows for the next reader are one kernel (`outnorm_residual`)."""
+    prompt_capturable = True
+    supports_append = True
+    reads_stream = True                  # the first block of a stack takes the embedding rows in the activation dtype
+
+    def __init__(self, mixer, feed_forward, mixer_norm, ffn_norm=None):
+        if (feed_forward is None) != (ffn_norm is None):
+            raise ValueError("OutputNormBlock: a feed-forward and its norm come together")
+        for norm in (mixer_norm, ffn_norm):
+            if norm is not None and getattr(norm, "fused_kind", None) != "rms":
+                raise ValueError("OutputNormBlock: its norms are RMS norms")
+        self.mixer, self.feed_forward, self.mixer_norm, self.ffn_norm = mixer, feed_forward, mixer_norm, ffn_norm
+
+    def children(self):
+        return [p for p in (self.mixer, self.mixer_norm, self.feed_forward, self.ffn_norm) if p is not None]
+
+    def state_spec(self):
+        return self.mixer.state_spec()
+
+    @staticmethod
+    def _sum(rt, h, y, norm, reader):
+        """h += norm(y); the rows for the next reader: its normed rows if it is an RMS norm, else the stream in the activation
+        dtype (None if another kind of norm comes next: its caller applies it)."""
+        fuse = getattr(reader, "fused_kind", None) == "rms"
+        if reader is not None and not fuse:
+            n = None
+        elif reader is None and rt.dtype == torch.float32:
+            n = h
+        else:
+            n = torch.empty(h.shape, dtype=rt.dtype, device=h.device)
+        kernels.outnorm_residual(h, _terms(y), norm.weight, norm.eps, n_out=None if n is h else n,
+                                 w_next=reader.weight if fuse else None, eps_next=reader.eps if fuse else 0.0)
+        return n
+
+    def forward(self, rt, batch, h, n, state, next_norm):
+        if h.dtype != torch.float32:
+            raise ValueError("OutputNormBlock works on a float32 residual stream (ModelDefinition.residual_float32)")
+        batch.partial_sums_ok = False
+        y = self.mixer.forward(rt, batch, n, state)
+        if self.feed_forward is None:
+            return h, self._sum(rt, h, y, self.mixer_norm, next_norm)
+        n = self._sum(rt, h, y, self.mixer_norm, None)
+        return h, self._sum(rt, h, self.feed_forward.forward(rt, batch, n), self.ffn_norm, next_norm)
+
+
 class HyperBlock(Block):
     """Two sublayers one after the other on hyper-connected streams X [rows, S, width] (float32).  Each sublayer f with its
     norm reads u = sum_s a_s X_s and is written back as X_t <- sum_s M[s, t] X_s + c_t f(norm(u)).  `input_norm` and
@@ -294,5 +345,6 @@ register_part("mixer", "side_by_side", SideBySide)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "postnorm", PostNormBlock)
+register_part("block", "outnorm", OutputNormBlock)
 register_part("block", "hyper", HyperBlock)
 register_part("block", "loop_entry", LoopEntry)

@@ -112,6 +112,24 @@ class PairedRotary(Position):
         return self._rate
 
 
+class WavelengthRotary(PairedRotary):
+    """`PairedRotary` whose rates are rescaled for a longer context by their wavelength l = 2 pi / f alone: pairs with
+    l < original / high keep their rate, pairs with l > original / low turn at f / factor, and between the two the rate is
+    (1 - s) f / factor + s f with s = (original / l - low) / (high - low).  Sine and cosine keep their magnitude."""
+
+    def __init__(self, dims, theta, factor, low, high, original):
+        import math
+
+        super().__init__(dims, theta)
+        for i, f in enumerate(self.rates):
+            wave = 2.0 * math.pi / f
+            if wave > original / low:
+                self.rates[i] = f / factor
+            elif wave >= original / high:
+                s = (original / wave - low) / (high - low)
+                self.rates[i] = (1.0 - s) * f / factor + s * f
+
+
 class NoPosition(Position):
     """No position encoding: the head vectors are left unrotated."""
     prompt_capturable = True
@@ -122,4 +140,5 @@ class NoPosition(Position):
 register_part("position", "rotary", Rotary)
 register_part("position", "none", NoPosition)
 register_part("position", "paired_rotary", PairedRotary)
+register_part("position", "wavelength_rotary", WavelengthRotary)
 register_part("position", "partial_yarn_rotary", PartialYarnRotary)
