@@ -617,6 +617,25 @@ def kofadra_config(size, vocab=VOCAB):
                 streams=4, layers=[delta, att] * 3, loop=dict(start=2, stop=4, times=2))
 
 
+def mogilorn_config(size, vocab=VOCAB):
+    """For `--compare mogilorn`: eight layers of the Mogilorn decoder at the same width, heads and feed-forward width as the Narasun
+    and the Relilix model above: an attention (scores capped at 30, mixed values, rates rescaled from 4,096 positions), a matrix
+    memory (Narasun's heads), a latent attention (Relilix's heads and latents, a window of 1,024 tokens), an attention, twice over;
+    plain feed-forwards."""
+    z = COMPARE_SIZES[size]
+    mlp = dict(kind="dense", ff=z["ff"])
+    scaling = dict(factor=4.0, low=1.0, high=4.0, original=4096)
+    att = dict(type="attention", mlp=mlp, mixer=dict(
+        heads=z["heads"], kv_heads=z["kv_heads"], dim=z["head"], vdim=z["head"], scale=z["head"] ** -0.5, softcap=30.0, v_mix=True,
+        rot=dict(dims=z["head"], base=1000000.0, scaling=scaling)))
+    mem = dict(type="mlstm", mlp=mlp, mixer=dict(heads=z["mem_heads"], dim=z["mem_dim"], vdim=z["mem_vdim"], gate_cap=15.0))
+    lat = dict(type="latent_attention", mlp=mlp, mixer=dict(
+        heads=z["heads"], dim=z["head"], rot_dim=32, vdim=z["head"], kv_rank=z["width"] // 4, scale=(z["head"] + 32) ** -0.5,
+        rot=dict(dims=32, base=1000000.0), mask=dict(size=1024)))
+    return dict(architecture="Mogilorn", vocab=vocab, width=z["width"], norm=dict(eps=1e-6), embedding=dict(scale=z["width"] ** 0.5),
+                layers=[att, mem, lat, att] * 2)
+
+
 def latent_decode_table(pk, device="cuda:0", cases=((8, 16, 256, 32), (128, 16, 256, 32), (64, 32, 512, 32)), held=2048):
     """`--latent-table`: the single-token latent attention alone, in its tensor-core and its CUDA-core form: `B` sequences
     that hold `held` tokens, `H` heads over latents of `KR` + `R` channels, random bfloat16 entries in pages laid out in
@@ -732,7 +751,8 @@ def _kernel_rows(torch, model, prompt_len, batch, vocab):
 def compare_designs(which, sizes, prompt_len, batch, steps, pk, tables):
     """Prefill and decode throughput of a design beside the closest earlier one at equal size, random weights: the
     Narasun decoder beside an LFM3 decoder, the Fozedra and the Maferax decoder beside the Narasun decoder, the Relilix
-    decoder beside the Maferax decoder, the Kofadra decoder beside the Narasun and the Maferax decoder."""
+    decoder beside the Maferax decoder, the Kofadra decoder beside the Narasun and the Maferax decoder, the Mogilorn decoder
+    beside the Narasun and the Relilix decoder."""
     import torch
 
     from catena_models_b200.api import Model
@@ -747,6 +767,7 @@ def compare_designs(which, sizes, prompt_len, batch, steps, pk, tables):
         pairs = {"narasun": (("Narasun", narasun_config), ("LFM3", lfm3_like_config)),
                  "fozedra": (("Fozedra", fozedra_config), ("Narasun", narasun_config)),
                  "maferax": (("Maferax", maferax_config), ("Narasun", narasun_config)),
+                 "mogilorn": (("Mogilorn", mogilorn_config), ("Narasun", narasun_config), ("Relilix", relilix_config)),
                  "relilix": (("Relilix", relilix_config), ("Maferax", maferax_config)),
                  "kofadra": (("Kofadra", kofadra_config), ("Narasun", narasun_config), ("Maferax", maferax_config))}[which]
         for name, cfg in ((n, make(size, vocab)) for n, make in pairs):
@@ -790,10 +811,10 @@ def main():
                     help="time the prompt-attention kernels alone at 2,048, 4,096 and 16,384 tokens and print the table")
     ap.add_argument("--latent-table", action="store_true",
                     help="instead of the JSON line: time the single-token latent attention alone, tensor-core and CUDA-core form")
-    ap.add_argument("--compare", default=None, choices=["narasun", "fozedra", "maferax", "relilix", "kofadra"],
+    ap.add_argument("--compare", default=None, choices=["narasun", "fozedra", "maferax", "relilix", "kofadra", "mogilorn"],
                     help="instead of the JSON line: prompt and decode throughput of that design beside the closest earlier "
                          "one at equal size (random weights: Narasun beside LFM3, Fozedra and Maferax beside Narasun, Relilix beside "
-                         "Maferax, Kofadra beside Narasun and Maferax), as a table")
+                         "Maferax, Kofadra beside Narasun and Maferax, Mogilorn beside Narasun and Relilix), as a table")
     ap.add_argument("--compare-sizes", default="1024,2048", help="widths of `--compare`")
     ap.add_argument("--compare-kernels", action="store_true", help="with `--compare`: also each model's kernel tables")
     ap.add_argument("--print-config", action="store_true",

@@ -236,6 +236,25 @@ def test_replay_of_a_kofadra_model(tmp_path, name, dtype):
     _replay_whole_tail_and_together(tmp_path, folder, V, reqs, exact, exact, dtype)
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "M"])
+def test_replay_of_a_mogilorn_model(tmp_path, name, dtype):
+    """The seventh architecture through the same program, on the same schedule (windows whose edge passes over prompts and over
+    decoded tokens, memories, mixed values); bfloat16 as for the fifth."""
+    import plain_mogilorn
+    import tiny_mogilorn
+
+    folder = tiny_mogilorn.make_folder(tmp_path, name, seed=7)
+    cfg, tensors = tiny_mogilorn.load_plain(folder)
+    V = cfg["vocab"]
+    reqs = {k: tiny_mogilorn.prompt(n, V, seed=ord(k)) for k, n in {"a": 1, "b": 70, "c": 135, "d": 90}.items()}
+    if dtype == "bfloat16":
+        _replay_whole_tail_and_together(tmp_path, folder, V, reqs, None, None, dtype, against_library=True)
+        return
+    exact = {k: plain_mogilorn.forward(t, tensors, cfg)[0] for k, t in reqs.items()}
+    _replay_whole_tail_and_together(tmp_path, folder, V, reqs, exact, exact, dtype)
+
+
 def _library_steps(folder, dtype, steps, max_tokens):
     """The same schedule through the library's engine in this process: {step: logits of its wanted places}."""
     from catena_models_b200.api import Model
