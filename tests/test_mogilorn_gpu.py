@@ -133,7 +133,7 @@ def test_prompt_then_token_by_token(folders, plains, name, dtype):
     check(run_alone(engine, tokens, [1]), ref, dtype)
 
 
-@pytest.mark.parametrize("name", ["A", "B", "C", "M"])
+@pytest.mark.parametrize("name", ["A", "B", "C", "M", "W"])
 def test_portions_of_several_sizes(folders, plains, name):
     engine = model_for(folders, name, "float32").engine
     tokens = tiny.prompt(200, tiny.ALL[name]["vocab"], 3)

@@ -92,6 +92,14 @@ TINY_L = model(120, 64, 1e-6, 1.5, [
     latent(1, 96, 32, 72, 40, 800, 0.09, 10000.0, 64),
     attention(1, 1, 128, 64, 0.09, None, rot(128, 10000.0), 40.0, True)])
 
+# W: heads beyond the tensor-core kernels, latents of many channels, more heads than a block of the latent kernels takes
+TINY_W = model(130, 96, 1e-5, 1.0, [
+    attention(2, 1, 160, 144, 0.08, 80, rot(120, 5000.0), 12.0, True),
+    latent(2, 112, 32, 136, 200, 90, 0.08, 700.0, 64),
+    mlstm(2, 144, 40, 6.0, 64),
+    latent(19, 8, 16, 24, 264, 37, 0.2, 700.0, None),
+    attention(8, 1, 20, 144, 0.2, 64, rot(20, 5000.0, (2.0, 1.0, 2.0, 128.0)), 7.0, True)])
+
 # one mechanism at a time
 ONLY_ATTENTION = model(64, 32, 1e-6, 1.0, [attention(4, 2, 16, 24, 0.3, None, rot(12, 100.0, (4.0, 1.0, 4.0, 60.0)), 3.0)])
 ONLY_MIX = model(64, 32, 1e-6, 1.0, [attention(2, 1, 16, 16, 0.3, None, None, None, True), attention(2, 1, 16, 16, 0.3, None, None, None, True)])
@@ -99,7 +107,7 @@ ONLY_MLSTM = model(64, 32, 1e-6, 1.0, [mlstm(4, 16, 24, 5.0, None)])
 ONLY_LATENT = model(64, 32, 1e-6, 1.0, [latent(4, 12, 8, 16, 24, 24, 0.3, 100.0, None)])
 ONLY_FF = model(64, 24, 1e-6, 1.0, [latent(1, 8, 0, 8, 8, 1, 0.3, 10.0, 88)])            # a window of the present token alone
 
-ALL = {"A": TINY_A, "B": TINY_B, "C": TINY_C, "M": TINY_M, "L": TINY_L, "attention": ONLY_ATTENTION, "mix": ONLY_MIX,
+ALL = {"A": TINY_A, "B": TINY_B, "C": TINY_C, "M": TINY_M, "L": TINY_L, "W": TINY_W, "attention": ONLY_ATTENTION, "mix": ONLY_MIX,
        "mlstm": ONLY_MLSTM, "latent": ONLY_LATENT, "ff": ONLY_FF}
 
 
