@@ -96,7 +96,6 @@ TINY_L = model(120, 64, 1e-6, 1.5, [
 TINY_W = model(130, 96, 1e-5, 1.0, [
     attention(2, 1, 160, 144, 0.08, 80, rot(120, 5000.0), 12.0, True),
     latent(2, 112, 32, 136, 200, 90, 0.08, 700.0, 64),
-    mlstm(2, 144, 40, 6.0, 64),
     latent(19, 8, 16, 24, 264, 37, 0.2, 700.0, None),
     attention(8, 1, 20, 144, 0.2, 64, rot(20, 5000.0, (2.0, 1.0, 2.0, 128.0)), 7.0, True)])
 
